@@ -11,7 +11,8 @@
 //
 // decay_attention: one block per (row, head, slice of the value entries); the slice's part of the state stays in
 // shared memory over the row's chunks and goes back to the request's slot at the end.
-// gated_rms_norm:  out = rmsnorm(o over all heads) * w * sigmoid(gate), one block per token.
+// gated_rms_norm:  out = rmsnorm(o over all heads) * w * sigmoid(gate), one block per token; or, with the gate first,
+//                  out = rmsnorm(o * silu(gate)) * w; the mean is taken over the row or over equal parts of it.
 #include "common.cuh"
 
 namespace {
@@ -19,6 +20,12 @@ constexpr int C = 32;            // tokens of a chunk
 constexpr int THREADS = 256;
 
 __device__ __forceinline__ float act_silu(float z) { return z / (1.f + expf(-z)); }
+
+// An entry behind the norm (scale: 1 / rms times the weight): times sigmoid(gate), or times silu(gate) where the gate came first.
+template <bool FIRST>
+__device__ __forceinline__ float gated_entry(float x, float gate, float scale) {
+  return x * scale * (FIRST ? act_silu(gate) : 1.f / (1.f + expf(-gate)));
+}
 
 template <typename T>
 __global__ void __launch_bounds__(THREADS)
@@ -436,36 +443,38 @@ size_t chunk_state_smem(int dk, int dvs) {
 }
 int chunk_slice(int dv) { return dv <= 64 ? dv : 64; }
 
-template <typename T>
-__global__ void gated_rms_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, int gate_stride,
+template <typename T, typename TG, bool FIRST>
+__global__ void gated_rms_norm_kernel(const float* __restrict__ o, const TG* __restrict__ gate, int gate_stride,
                                       const float* __restrict__ w, T* __restrict__ out, int n, float eps) {
   __shared__ float scratch[34];
   const int t = blockIdx.x;
   const float* x = o + (size_t)t * n;
+  const TG* gt = gate + (size_t)t * gate_stride;
   float ss = 0.f;
-  for (int i = threadIdx.x; i < n; i += blockDim.x) ss += x[i] * x[i];
+  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    const float v = FIRST ? x[i] * act_silu(to_f32<TG>(gt[i])) : x[i];
+    ss += v * v;
+  }
   ss = block_sum(ss, scratch);
   const float inv = 1.f / sqrtf(ss / (float)n + eps);
-  for (int i = threadIdx.x; i < n; i += blockDim.x) {
-    const float g = to_f32<T>(gate[(size_t)t * gate_stride + i]);
-    out[(size_t)t * n + i] = from_f32<T>(x[i] * inv * w[i] * (1.f / (1.f + expf(-g))));
-  }
+  for (int i = threadIdx.x; i < n; i += blockDim.x) out[(size_t)t * n + i] = from_f32<T>(gated_entry<FIRST>(x[i], to_f32<TG>(gt[i]), inv * w[i]));
 }
 
 // The same with the statistics taken per group of `group` consecutive entries (a head): one warp per group.
-template <typename T>
-__global__ void gated_group_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, int gate_stride,
+template <typename T, typename TG, bool FIRST>
+__global__ void gated_group_norm_kernel(const float* __restrict__ o, const TG* __restrict__ gate, int gate_stride,
                                         const float* __restrict__ w, T* __restrict__ out, int n, int group, float eps) {
   const int t = blockIdx.x, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
   const float* x = o + (size_t)t * n;
+  const TG* gt = gate + (size_t)t * gate_stride;
   for (int g0 = (threadIdx.x >> 5) * group; g0 < n; g0 += warps * group) {
     float ss = 0.f;
-    for (int i = lane; i < group; i += 32) ss += x[g0 + i] * x[g0 + i];
-    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)group + eps);
     for (int i = g0 + lane; i < g0 + group; i += 32) {
-      const float g = to_f32<T>(gate[(size_t)t * gate_stride + i]);
-      out[(size_t)t * n + i] = from_f32<T>(x[i] * inv * w[i] * (1.f / (1.f + expf(-g))));
+      const float v = FIRST ? x[i] * act_silu(to_f32<TG>(gt[i])) : x[i];
+      ss += v * v;
     }
+    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)group + eps);
+    for (int i = g0 + lane; i < g0 + group; i += 32) out[(size_t)t * n + i] = from_f32<T>(gated_entry<FIRST>(x[i], to_f32<TG>(gt[i]), inv * w[i]));
   }
 }
 
@@ -511,24 +520,27 @@ extern "C" int dk_decay_attention(const void* src, int src_stride, int q_off, in
 
 // group: the entries whose root mean square is taken together (n: the whole row; a divisor of n: one head at a time)
 extern "C" int dk_gated_rms_norm(const float* o, const void* gate, int gate_stride, const float* w, void* out, int T_, int n, float eps,
-                                 int group, int dtype, cudaStream_t stream) {
+                                 int group, int gate_first, int gate_dtype, int dtype, cudaStream_t stream) {
   if (T_ == 0) return 0;
   DK_REQUIRE(T_ > 0 && n > 0 && gate_stride >= n, "gated_rms_norm: bad sizes T=%d n=%d stride=%d", T_, n, gate_stride);
   DK_REQUIRE(group > 0 && n % group == 0, "gated_rms_norm: groups of %d entries do not divide a row of %d", group, n);
   const int threads = n >= 2048 ? 256 : 128;
-  if (group != n) {
-    if (dtype == DK_F32)
-      gated_group_norm_kernel<float><<<T_, threads, 0, stream>>>(o, (const float*)gate, gate_stride, w, (float*)out, n, group, eps);
-    else if (dtype == DK_BF16)
-      gated_group_norm_kernel<__nv_bfloat16><<<T_, threads, 0, stream>>>(o, (const __nv_bfloat16*)gate, gate_stride, w, (__nv_bfloat16*)out, n, group, eps);
-    else DK_REQUIRE(false, "gated_rms_norm: unknown dtype %d", dtype);
-    return dk_check_launch("gated_rms_norm");
-  }
-  if (dtype == DK_F32)
-    gated_rms_norm_kernel<float><<<T_, threads, 0, stream>>>(o, (const float*)gate, gate_stride, w, (float*)out, n, eps);
-  else if (dtype == DK_BF16)
-    gated_rms_norm_kernel<__nv_bfloat16><<<T_, threads, 0, stream>>>(o, (const __nv_bfloat16*)gate, gate_stride, w, (__nv_bfloat16*)out, n, eps);
-  else DK_REQUIRE(false, "gated_rms_norm: unknown dtype %d", dtype);
+#define LAUNCH(T, TG, FIRST)                                                                                                      \
+  do {                                                                                                                            \
+    if (group != n) gated_group_norm_kernel<T, TG, FIRST><<<T_, threads, 0, stream>>>(o, (const TG*)gate, gate_stride, w, (T*)out, n, group, eps); \
+    else gated_rms_norm_kernel<T, TG, FIRST><<<T_, threads, 0, stream>>>(o, (const TG*)gate, gate_stride, w, (T*)out, n, eps);     \
+  } while (0)
+#define BOTH(T, TG)                      \
+  do {                                   \
+    if (gate_first) LAUNCH(T, TG, true); \
+    else LAUNCH(T, TG, false);           \
+  } while (0)
+  if (dtype == DK_F32 && gate_dtype == DK_F32) BOTH(float, float);
+  else if (dtype == DK_BF16 && gate_dtype == DK_BF16) BOTH(__nv_bfloat16, __nv_bfloat16);
+  else if (dtype == DK_BF16 && gate_dtype == DK_F32) BOTH(__nv_bfloat16, float);
+  else DK_REQUIRE(false, "gated_rms_norm: unsupported dtypes gate=%d out=%d", gate_dtype, dtype);
+#undef BOTH
+#undef LAUNCH
   return dk_check_launch("gated_rms_norm");
 }
 

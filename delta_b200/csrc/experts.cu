@@ -4,7 +4,8 @@
 //                   from rows [g (F) | u (F)] (limit < 0: nothing is clamped);
 //   router          per token the router's logits z = W x in 32 bit, the `top` largest of the E experts' logits (the lowest
 //                   index among equals) and the softmax over the chosen logits only (router_topk: the choice alone, from
-//                   logits that are there already);
+//                   logits that are there already); or scores (sigmoid, or the softmax over all E) with a correction that
+//                   joins the choice only, optionally restricted to the best groups of neighbouring experts;
 //   experts_align   sorts the (token, choice) slots by expert into tiles of `tile_m` rows that each belong to one expert
 //                   (every expert's rows padded to whole tiles with -1), so that the products run as one launch and
 //                   nothing about the routing is read on the host;
@@ -14,7 +15,8 @@
 //                   the slot's weight first, which is what an expert that reads weight * x gets).  Second product: rows are read in the
 //                   sorted order and the result goes to the slot's own place, in 32 bit;
 //   experts_combine out[t] = sum_j weight[t][j] * z[t*top + j]  (+ sigmoid(gate logit of t) * shared[t]), summed in 32 bit in
-//                   the order of the choices, so the result does not depend on what else is in the batch.
+//                   the order of the choices, so the result does not depend on what else is in the batch.  A choice from
+//                   `identity_from` on has no matrices: what it adds is weight * x[t], the layer's own input.
 //
 // The products run on the tensor cores for bfloat16 (warp-level MMA, 32-bit accumulation) and on the FMA units in 32 bit
 // (and for bfloat16 rows whose length is no multiple of 8).
@@ -103,7 +105,42 @@ __device__ void pick_top(float* z, int E, int top, int* __restrict__ choice, flo
   }
 }
 
-// The choice by sigmoid scores: `pick` [E] holds score + correction and is used up, `score` [E] the scores s = sigmoid(z).  The
+// Only the `keep` best of `count` equal groups of neighbouring experts can be chosen: a group's score is its largest pick (the
+// lowest group among equals), the picks of the other groups become -inf.  `best` [count] is the warp's own memory.
+__device__ void keep_groups(float* pick, float* best, int E, int count, int keep, int lane) {
+  const int per = E / count;
+  for (int g = lane; g < count; g += 32) {
+    float m = -INFINITY;
+    for (int i = 0; i < per; ++i) m = fmaxf(m, pick[g * per + i]);
+    best[g] = m;
+  }
+  __syncwarp();
+  for (int j = 0; j < keep; ++j) {
+    float bv = -INFINITY;
+    int bg = 0x7fffffff;
+    for (int g = lane; g < count; g += 32)
+      if (best[g] > bv) {
+        bv = best[g];
+        bg = g;
+      }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+      const int og = __shfl_xor_sync(0xffffffffu, bg, o);
+      if (ov > bv || (ov == bv && og < bg)) {
+        bv = ov;
+        bg = og;
+      }
+    }
+    if (lane == 0 && bg < count) best[bg] = -INFINITY;      // kept (scores are finite)
+    __syncwarp();
+  }
+  for (int e = lane; e < E; e += 32)
+    if (best[e / per] != -INFINITY) pick[e] = -INFINITY;
+  __syncwarp();
+}
+
+// The choice by scores: `pick` [E] holds score + correction and is used up, `score` [E] the scores s.  The
 // `top` largest of pick are chosen (the lowest index among equals); a chosen expert's weight is its score without the
 // correction, divided by the sum of the chosen scores (+ 1e-20) when `normalize`, times `scale`.
 __device__ void pick_top_scored(float* pick, const float* score, int E, int top, float scale, int normalize, int* __restrict__ choice,
@@ -169,8 +206,8 @@ template <typename T, bool VEC>
 __global__ void __launch_bounds__(ROUTER_WARPS * 32)
 router_kernel(const T* __restrict__ x, const T* __restrict__ w, float* __restrict__ logits, int* __restrict__ choice,
               float* __restrict__ weight, int T_, int d, int n_rows, int E, int top, int tpb, const float* __restrict__ correction,
-              float route_scale, int scored) {
-  extern __shared__ float zs[];      // [tpb][n_rows] (scored: and [tpb][E] behind them)
+              float route_scale, int scored, int groups, int keep) {
+  extern __shared__ float zs[];      // [tpb][n_rows] (scored: and [tpb][E] behind them; with groups: and [tpb][groups])
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int local = warp % tpb, share = warp / tpb, sharers = ROUTER_WARPS / tpb;
   const int t = blockIdx.x * tpb + local;
@@ -215,16 +252,25 @@ router_kernel(const T* __restrict__ x, const T* __restrict__ w, float* __restric
   }
   __syncthreads();
   if (!live || share != 0) return;
-  if (scored) {      // sigmoid scores; the correction joins the choice only
+  if (scored) {      // scores; the correction joins the choice only
     float* score = zs + (size_t)tpb * n_rows + (size_t)local * E;
+    float largest = -INFINITY, sum = 1.f;
+    if (scored >= 3) {      // the softmax over all experts
+      for (int e = lane; e < E; e += 32) largest = fmaxf(largest, z[e]);
+      largest = warp_max(largest);
+      sum = 0.f;
+      for (int e = lane; e < E; e += 32) sum += expf(z[e] - largest);
+      sum = warp_sum(sum);
+    }
     for (int e = lane; e < E; e += 32) {
-      const float sc = 1.f / (1.f + expf(-z[e]));
+      const float sc = scored >= 3 ? expf(z[e] - largest) / sum : 1.f / (1.f + expf(-z[e]));
       score[e] = sc;
-      // without a correction the logits themselves are compared: the same order, and no ties where the sigmoid saturates
+      // without a correction the logits themselves are compared: the same order, and no ties where the score saturates
       if (correction != nullptr) z[e] = sc + correction[e];
     }
     __syncwarp();
-    pick_top_scored(z, score, E, top, route_scale, scored == 1, choice + (size_t)t * top, weight + (size_t)t * top, lane);
+    if (groups > 0) keep_groups(z, zs + (size_t)tpb * (n_rows + E) + (size_t)local * groups, E, groups, keep, lane);
+    pick_top_scored(z, score, E, top, route_scale, scored & 1, choice + (size_t)t * top, weight + (size_t)t * top, lane);
   } else {
     pick_top(z, E, top, choice + (size_t)t * top, weight + (size_t)t * top, lane);
   }
@@ -514,15 +560,20 @@ __global__ void experts_gather_kernel(const __nv_bfloat16* __restrict__ x, const
   }
 }
 
-template <typename T>
+template <typename T, typename TX>
 __global__ void experts_combine_kernel(const float* __restrict__ z, const float* __restrict__ weight, int top, const T* __restrict__ shared,
-                                       const float* __restrict__ gate_logit, int gate_stride, T* __restrict__ out, int d) {
+                                       const float* __restrict__ gate_logit, int gate_stride, T* __restrict__ out, int d,
+                                       const TX* __restrict__ x, const int* __restrict__ choice, int identity_from) {
   const int t = blockIdx.x;
   float gate = 0.f;
   if (shared != nullptr) gate = gate_logit != nullptr ? 1.f / (1.f + expf(-gate_logit[(size_t)t * gate_stride])) : 1.f;
   for (int i = threadIdx.x; i < d; i += blockDim.x) {
     float a = 0.f;
-    for (int j = 0; j < top; ++j) a = fmaf(weight != nullptr ? weight[(size_t)t * top + j] : 1.f, z[((size_t)t * top + j) * d + i], a);
+    for (int j = 0; j < top; ++j) {
+      const bool through = x != nullptr && choice[(size_t)t * top + j] >= identity_from;
+      const float v = through ? to_f32<TX>(x[(size_t)t * d + i]) : z[((size_t)t * top + j) * d + i];
+      a = fmaf(weight != nullptr ? weight[(size_t)t * top + j] : 1.f, v, a);
+    }
     if (shared != nullptr) a = fmaf(gate, to_f32<T>(shared[(size_t)t * d + i]), a);
     out[(size_t)t * d + i] = from_f32<T>(a);
   }
@@ -564,20 +615,25 @@ extern "C" int dk_router_topk(const float* logits, int ld, int* choice, float* w
 
 // scored == 0: the softmax over the chosen logits.  scored == 1: sigmoid scores, `correction` [E] (or null) added for the choice
 // only, weights = chosen scores / their sum * route_scale.  scored == 2: the same with weights = chosen scores * route_scale.
+// scored == 3, 4: as 1, 2 with the softmax over all E logits as scores.  groups > 0 (scored only): the experts form that many
+// equal groups of neighbours, of which the `keep` with the largest score + correction can be chosen from.
 extern "C" int dk_router(const void* x, const void* w, float* logits, int* choice, float* weight, int T_, int d, int n_rows, int E, int top,
-                         const float* correction, float route_scale, int scored, int dtype, cudaStream_t stream) {
+                         const float* correction, float route_scale, int scored, int groups, int keep, int dtype, cudaStream_t stream) {
   if (T_ == 0) return 0;
   DK_REQUIRE(T_ > 0 && d > 0 && E > 0 && top > 0 && top <= E && n_rows >= E, "router: bad sizes T=%d d=%d E=%d top=%d rows=%d", T_, d, E, top, n_rows);
   DK_REQUIRE(top <= MAX_TOP, "router: %d choices a token are above the %d this kernel takes", top, MAX_TOP);
+  DK_REQUIRE(scored >= 0 && scored <= 4, "router: unknown scoring %d", scored);
+  DK_REQUIRE(groups == 0 || (scored > 0 && groups > 0 && E % groups == 0 && keep >= 1 && keep <= groups && keep * (E / groups) >= top),
+             "router: %d of %d groups of %d experts do not hold %d choices", keep, groups, E, top);
   // few tokens: one token a block, its rows shared by the block's warps; many: eight tokens a block
-  const int groups = (n_rows + ROUTER_ROWS - 1) / ROUTER_ROWS;
+  const int row_groups = (n_rows + ROUTER_ROWS - 1) / ROUTER_ROWS;
   int tpb = ROUTER_WARPS;
-  while (tpb > 1 && (ROUTER_WARPS / tpb < groups) && (long long)T_ * (ROUTER_WARPS / tpb) < 16LL * dk_sm_count()) tpb /= 2;
-  const size_t smem = (size_t)tpb * (n_rows + (scored ? E : 0)) * sizeof(float);
+  while (tpb > 1 && (ROUTER_WARPS / tpb < row_groups) && (long long)T_ * (ROUTER_WARPS / tpb) < 16LL * dk_sm_count()) tpb /= 2;
+  const size_t smem = (size_t)tpb * (n_rows + (scored ? E : 0) + groups) * sizeof(float);
   DK_REQUIRE(smem <= 48 * 1024, "router: %d logits a token do not fit the shared memory", n_rows);
   const int blocks = (T_ + tpb - 1) / tpb;
   const bool vec = d % 8 == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)w % 16) == 0;
-#define LAUNCH(T, V) router_kernel<T, V><<<blocks, ROUTER_WARPS * 32, smem, stream>>>((const T*)x, (const T*)w, logits, choice, weight, T_, d, n_rows, E, top, tpb, correction, route_scale, scored)
+#define LAUNCH(T, V) router_kernel<T, V><<<blocks, ROUTER_WARPS * 32, smem, stream>>>((const T*)x, (const T*)w, logits, choice, weight, T_, d, n_rows, E, top, tpb, correction, route_scale, scored, groups, keep)
   if (dtype == DK_F32) {
     if (vec) LAUNCH(float, true);
     else LAUNCH(float, false);
@@ -656,15 +712,19 @@ extern "C" int dk_experts_gather(const void* x, const int* sorted, int top, void
 }
 
 extern "C" int dk_experts_combine(const float* z, const float* weight, int top, const void* shared, const float* gate_logit,
-                                  int gate_stride, void* out, int T_, int d, int dtype, cudaStream_t stream) {
+                                  int gate_stride, void* out, int T_, int d, const void* x, const int* choice, int identity_from,
+                                  int x_dtype, int dtype, cudaStream_t stream) {
   if (T_ == 0) return 0;
   DK_REQUIRE(T_ > 0 && d > 0 && top > 0, "experts_combine: bad sizes T=%d d=%d top=%d", T_, d, top);
+  DK_REQUIRE(x == nullptr || (choice != nullptr && identity_from >= 0), "experts_combine: an input is given without the choices");
   const int threads = d >= 1024 ? 256 : 128;
-  if (dtype == DK_F32)
-    experts_combine_kernel<float><<<T_, threads, 0, stream>>>(z, weight, top, (const float*)shared, gate_logit, gate_stride, (float*)out, d);
-  else if (dtype == DK_BF16)
-    experts_combine_kernel<__nv_bfloat16><<<T_, threads, 0, stream>>>(z, weight, top, (const __nv_bfloat16*)shared, gate_logit, gate_stride,
-                                                                      (__nv_bfloat16*)out, d);
+#define LAUNCH(T, TX)                                                                                                             \
+  experts_combine_kernel<T, TX><<<T_, threads, 0, stream>>>(z, weight, top, (const T*)shared, gate_logit, gate_stride, (T*)out, d, \
+                                                            (const TX*)x, choice, identity_from)
+  if (dtype == DK_F32 && x_dtype == DK_F32) LAUNCH(float, float);
+  else if (dtype == DK_F32 && x_dtype == DK_BF16) LAUNCH(float, __nv_bfloat16);
+  else if (dtype == DK_BF16 && x_dtype == DK_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);
+#undef LAUNCH
   else DK_REQUIRE(false, "experts_combine: unknown dtype %d", dtype);
   return dk_check_launch("experts_combine");
 }

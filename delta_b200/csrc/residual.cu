@@ -2,10 +2,10 @@
 //
 //   embedding_pair   x = table[token] * scale + pair_table[hash(previous token, token)]
 //                    (the previous token of a portion's first token comes from the request's state;
-//                    a sequence's first token takes the pair table's last row);
+//                    a sequence's first token takes the pair table's last row), then, if asked for, x = norm(x) * w + b;
 //   remember_tokens  leaves every row's last token in that state;
 //   residual_norm    the step between two layers, in one pass over the stream:
-//                        x <- x + (y1 + y2)      what the last layer's sublayers gave (either may be absent)
+//                        x <- x + m (y1 + y2)    what the last layer's sublayers gave (either may be absent), times a constant
 //                        x <- x + e              a second 32-bit stream (the embedding output, at a re-entry)
 //                        x <- x + vec            one vector for all tokens
 //                    then out = norm(x) * w with the layer norm without bias, (x - mean) / sqrt(var + eps), var the
@@ -22,7 +22,9 @@ __global__ void embedding_pair_kernel(const int* __restrict__ tokens, const int*
                                       const int* __restrict__ row_q_start, const int* __restrict__ row_slot,
                                       const int* __restrict__ prev_state, const T* __restrict__ table, float scale,
                                       const T* __restrict__ pair_table, long long buckets, long long mul_prev, long long mul_cur,
-                                      float* __restrict__ X, float* __restrict__ E, T* __restrict__ R, int d, int vocab, int* err) {
+                                      float* __restrict__ X, float* __restrict__ E, T* __restrict__ R, const float* __restrict__ norm_w,
+                                      const float* __restrict__ norm_b, float eps, int kind, int d, int vocab, int* err) {
+  extern __shared__ __align__(16) float row_sm[];   // with a norm: d floats + 36
   const int t = blockIdx.x;
   const int tok = tokens[t];
   const bool bad = tok < 0 || tok >= vocab;
@@ -40,9 +42,31 @@ __global__ void embedding_pair_kernel(const int* __restrict__ tokens, const int*
     pair = pair_table + (size_t)b * d;
   }
   const T* src = table + (size_t)(bad ? 0 : tok) * d;
+  float mean = 0.f, inv = 1.f;
+  if (norm_w != nullptr) {
+    float* scratch = row_sm + d;
+    float sum = 0.f, ss = 0.f;
+    for (int i = threadIdx.x; i < d; i += blockDim.x) {
+      float v = bad ? 0.f : to_f32<T>(src[i]) * scale;
+      if (pair != nullptr) v += to_f32<T>(pair[i]);
+      row_sm[i] = v;
+      sum += v;
+    }
+    if (kind == 1) mean = block_sum(sum, scratch) / (float)d;
+    for (int i = threadIdx.x; i < d; i += blockDim.x) {
+      const float c = row_sm[i] - mean;
+      ss += c * c;
+    }
+    inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)d + eps);
+  }
   for (int i = threadIdx.x; i < d; i += blockDim.x) {
-    float v = bad ? 0.f : to_f32<T>(src[i]) * scale;
-    if (pair != nullptr) v += to_f32<T>(pair[i]);
+    float v;
+    if (norm_w != nullptr) {
+      v = (row_sm[i] - mean) * inv * norm_w[i] + (norm_b != nullptr ? norm_b[i] : 0.f);
+    } else {
+      v = bad ? 0.f : to_f32<T>(src[i]) * scale;
+      if (pair != nullptr) v += to_f32<T>(pair[i]);
+    }
     X[(size_t)t * d + i] = v;
     if (E != nullptr) E[(size_t)t * d + i] = v;
     if (R != nullptr) R[(size_t)t * d + i] = from_f32<T>(v);      // the stream in the compute type, for a first sublayer that reads it
@@ -58,7 +82,7 @@ __global__ void remember_tokens_kernel(const int* __restrict__ tokens, const int
 
 // One block per output row r (token tk = rows ? rows[r] : r); the settled row is kept in shared memory between the passes.
 template <typename T, typename TO>
-__global__ void residual_norm_kernel(float* __restrict__ X, const T* __restrict__ y1, const T* __restrict__ y2, const float* __restrict__ e,
+__global__ void residual_norm_kernel(float* __restrict__ X, const T* __restrict__ y1, const T* __restrict__ y2, float mult, const float* __restrict__ e,
                                      const float* __restrict__ vec, const float* __restrict__ w, const float* __restrict__ b,
                                      TO* __restrict__ out, const int* __restrict__ rows, int d, float eps, int kind, int write_back) {
   extern __shared__ __align__(16) float xs[];   // d floats + 33
@@ -72,7 +96,7 @@ __global__ void residual_norm_kernel(float* __restrict__ X, const T* __restrict_
     if (y1 != nullptr) {
       float u = to_f32<T>(y1[(size_t)tk * d + i]);
       if (y2 != nullptr) u += to_f32<T>(y2[(size_t)tk * d + i]);
-      v += u;
+      v = fmaf(mult, u, v);
     }
     if (e != nullptr) v += e[(size_t)tk * d + i];
     if (vec != nullptr) v += vec[i];
@@ -183,15 +207,19 @@ extern "C" int dk_normed_sum(const float* y1, const float* b1, const float* w1, 
 
 extern "C" int dk_embedding_pair(const int* tokens, const int* tok_row, const int* tok_pos, const int* row_q_start, const int* row_slot,
                                  int* prev_state, const void* table, float scale, const void* pair_table, long long buckets,
-                                 long long mul_prev, long long mul_cur, float* X, float* E, void* R, int T_, int d, int vocab, int dtype, int* err,
-                                 cudaStream_t stream) {
+                                 long long mul_prev, long long mul_cur, float* X, float* E, void* R, const float* norm_w, const float* norm_b,
+                                 float eps, int kind, int T_, int d, int vocab, int dtype, int* err, cudaStream_t stream) {
   if (T_ == 0) return 0;
   DK_REQUIRE(T_ > 0 && d > 0 && vocab > 0, "embedding_pair: bad sizes T=%d d=%d vocab=%d", T_, d, vocab);
   DK_REQUIRE(pair_table == nullptr || (buckets > 0 && prev_state != nullptr), "embedding_pair: a pair table needs buckets and the state of previous tokens");
+  DK_REQUIRE(norm_w == nullptr || d <= 12000, "embedding_pair: width %d is above the 12000 that a norm keeps in shared memory", d);
+  DK_REQUIRE(kind == 0 || kind == 1, "embedding_pair: unknown norm kind %d", kind);
   const int threads = d >= 1024 ? 256 : 128;
+  const size_t smem = norm_w != nullptr ? (size_t)(d + 36) * sizeof(float) : 0;
 #define LAUNCH(T)                                                                                                               \
-  embedding_pair_kernel<T><<<T_, threads, 0, stream>>>(tokens, tok_row, tok_pos, row_q_start, row_slot, prev_state, (const T*)table, \
-                                                        scale, (const T*)pair_table, buckets, mul_prev, mul_cur, X, E, (T*)R, d, vocab, err)
+  embedding_pair_kernel<T><<<T_, threads, smem, stream>>>(tokens, tok_row, tok_pos, row_q_start, row_slot, prev_state, (const T*)table, \
+                                                        scale, (const T*)pair_table, buckets, mul_prev, mul_cur, X, E, (T*)R, norm_w, \
+                                                        norm_b, eps, kind, d, vocab, err)
   if (dtype == DK_F32) LAUNCH(float);
   else if (dtype == DK_BF16) LAUNCH(__nv_bfloat16);
   else DK_REQUIRE(false, "embedding_pair: unknown dtype %d", dtype);
@@ -207,7 +235,7 @@ extern "C" int dk_remember_tokens(const int* tokens, const int* row_q_start, con
   return dk_check_launch("remember_tokens");
 }
 
-extern "C" int dk_residual_norm(float* X, const void* y1, const void* y2, const float* e, const float* vec, const float* w, const float* b,
+extern "C" int dk_residual_norm(float* X, const void* y1, const void* y2, float mult, const float* e, const float* vec, const float* w, const float* b,
                                 void* out, const int* rows, int n_rows, int d, float eps, int kind, int write_back, int y_dtype, int out_dtype,
                                 cudaStream_t stream) {
   if (n_rows == 0) return 0;
@@ -218,7 +246,7 @@ extern "C" int dk_residual_norm(float* X, const void* y1, const void* y2, const 
   const int threads = d >= 4096 ? 512 : (d >= 1024 ? 256 : 128);
   const size_t smem = (size_t)(d + 36) * sizeof(float);
 #define LAUNCH(T, TO)                                                                                                          \
-  residual_norm_kernel<T, TO><<<n_rows, threads, smem, stream>>>(X, (const T*)y1, (const T*)y2, e, vec, w, b, (TO*)out, rows, d, eps, \
+  residual_norm_kernel<T, TO><<<n_rows, threads, smem, stream>>>(X, (const T*)y1, (const T*)y2, mult, e, vec, w, b, (TO*)out, rows, d, eps, \
                                                                  kind, write_back)
   if (y_dtype == DK_F32 && out_dtype == DK_F32) LAUNCH(float, float);
   else if (y_dtype == DK_BF16 && out_dtype == DK_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);

@@ -62,6 +62,81 @@ __global__ void conv_state_kernel(const T* __restrict__ xin, int in_stride, floa
     if (j < taps - 1) st[(size_t)j * C + c] = v[j];
 }
 
+// The same for 2 to 4 taps, C a multiple of 8 and 16-byte aligned rows: a thread takes eight channels of CONV_TOKENS tokens that
+// follow one another and keeps the window of inputs in registers, so every input is read once per tile.
+// grid (ceil(tokens / CONV_TOKENS), ceil(C / 8 / blockDim))
+constexpr int CONV_TOKENS = 8;
+template <typename T, int TAPS>
+__global__ void conv_silu_vec_kernel(const T* __restrict__ xin, int in_stride, const float* __restrict__ w, const float* __restrict__ bias,
+                                     const float* __restrict__ conv_state, T* __restrict__ out, const int* __restrict__ tok_row,
+                                     const int* __restrict__ row_slot, const int* __restrict__ row_q_start, int tokens, int C, int act) {
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
+  if (c >= C) return;
+  const int t_from = blockIdx.x * CONV_TOKENS, t_to = min(t_from + CONV_TOKENS, tokens);
+  float wv[TAPS][8], b[8], win[TAPS - 1][8];
+#pragma unroll
+  for (int e = 0; e < 8; ++e) {
+    b[e] = bias ? bias[c + e] : 0.f;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) wv[j][e] = w[(size_t)(c + e) * TAPS + j];
+  }
+  int row = -1;
+  for (int t = t_from; t < t_to; ++t) {
+    if (tok_row[t] != row) {      // the first token of the tile, or of a row: the inputs before it
+      row = tok_row[t];
+      const int q0 = row_q_start[row];
+      const float* st = conv_state + (size_t)row_slot[row] * (TAPS - 1) * C;
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) {
+        const int k = t - q0 - (TAPS - 1) + j;
+        if (k >= 0) load8<T>(xin + (size_t)(q0 + k) * in_stride + c, win[j]);
+        else load8<float>(st + (size_t)(TAPS - 1 + k) * C + c, win[j]);
+      }
+    }
+    float x[8], o[8];
+    load8<T>(xin + (size_t)t * in_stride + c, x);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      float acc = b[e];
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) acc = fmaf(wv[j][e], win[j][e], acc);
+      acc = fmaf(wv[TAPS - 1][e], x[e], acc);
+      o[e] = act ? acc / (1.f + expf(-acc)) : acc;
+#pragma unroll
+      for (int j = 0; j + 1 < TAPS - 1; ++j) win[j][e] = win[j + 1][e];
+      win[TAPS - 2][e] = x[e];
+    }
+    store8<T>(out + (size_t)t * C + c, o);
+  }
+}
+
+// Every row brings one token: the convolution and the state's step in one kernel, one thread per (row, channel).
+template <typename T>
+__global__ void conv_step_kernel(const T* __restrict__ xin, int in_stride, const float* __restrict__ w, const float* __restrict__ bias,
+                                 float* __restrict__ conv_state, T* __restrict__ out, const int* __restrict__ row_slot,
+                                 const int* __restrict__ row_q_start, int C, int taps, const float* __restrict__ in_bias, int act) {
+  const int row = blockIdx.x;
+  const int c = blockIdx.y * blockDim.x + threadIdx.x;
+  if (c >= C) return;
+  const size_t t = (size_t)row_q_start[row];
+  float* st = conv_state + (size_t)row_slot[row] * (taps - 1) * C + c;
+  const float x = to_f32<T>(xin[t * in_stride + c]) + (in_bias ? in_bias[c] : 0.f);
+  const float* wc = w + (size_t)c * taps;
+  float v[MAX_TAPS];
+  float acc = bias ? bias[c] : 0.f;
+#pragma unroll
+  for (int j = 0; j < MAX_TAPS - 1; ++j)
+    if (j < taps - 1) {
+      v[j] = st[(size_t)j * C];
+      acc = fmaf(wc[j], v[j], acc);
+    }
+  acc = fmaf(wc[taps - 1], x, acc);
+  out[t * C + c] = from_f32<T>(act ? acc / (1.f + expf(-acc)) : acc);
+#pragma unroll
+  for (int j = 0; j < MAX_TAPS - 1; ++j)
+    if (j < taps - 1) st[(size_t)j * C] = j + 1 < taps - 1 ? v[j + 1] : x;
+}
+
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 
 // Block: 128 threads = (128 / P) channels x P lanes; lane p of a channel keeps the states n = p, p + P, ...
@@ -197,9 +272,9 @@ __global__ void scan_combine_kernel(const float* __restrict__ A_log, float* __re
 
 extern "C" int dk_conv_silu(const void* xin, int in_stride, const float* w, const float* bias, float* conv_state, void* out,
                             const int* tok_row, const int* row_slot, const int* row_q_start, const int* row_q_len, int T_,
-                            int rows, int C, int taps, const float* in_bias, int act, int dtype, cudaStream_t stream) {
+                            int rows, int C, int taps, const float* in_bias, int act, int single, int dtype, cudaStream_t stream) {
   // in_bias [C] (or null) is added to every input as it is read, not to the zeros before a request's first token;
-  // act 1: silu behind the convolution, 0: none
+  // act 1: silu behind the convolution, 0: none; single: every row brings one token (one kernel instead of two)
   if (T_ == 0) return 0;
   DK_REQUIRE(T_ > 0 && rows > 0 && C > 0 && in_stride >= C, "conv_silu: bad sizes T=%d rows=%d C=%d stride=%d", T_, rows, C, in_stride);
   DK_REQUIRE(taps >= 1 && taps <= MAX_TAPS, "conv_silu: %d taps; this kernel takes 1 to %d", taps, MAX_TAPS);
@@ -207,6 +282,34 @@ extern "C" int dk_conv_silu(const void* xin, int in_stride, const float* w, cons
   const int threads = C >= 256 ? 256 : 128;
   const dim3 g1(T_, (C + threads - 1) / threads), g2(rows, (C + threads - 1) / threads);
   DK_REQUIRE(g1.y <= 65535, "conv_silu: too many channels");
+  if (single && taps > 1) {
+#define STEP(T)                                                                                                                  \
+  conv_step_kernel<T><<<g2, threads, 0, stream>>>((const T*)xin, in_stride, w, bias, conv_state, (T*)out, row_slot, row_q_start, C, taps, \
+                                                  in_bias, act)
+    if (dtype == DK_F32) STEP(float);
+    else STEP(__nv_bfloat16);
+#undef STEP
+    return dk_check_launch("conv_silu");
+  }
+  if (taps >= 2 && taps <= 4 && in_bias == nullptr && C % 8 == 0 && in_stride % 8 == 0 && ((uintptr_t)xin % 16) == 0 && ((uintptr_t)out % 16) == 0 &&
+      ((uintptr_t)conv_state % 16) == 0) {
+    const dim3 gv((T_ + CONV_TOKENS - 1) / CONV_TOKENS, (C / 8 + 127) / 128);
+#define VEC(T, TAPS)                                                                                                              \
+  conv_silu_vec_kernel<T, TAPS><<<gv, 128, 0, stream>>>((const T*)xin, in_stride, w, bias, conv_state, (T*)out, tok_row, row_slot, row_q_start, \
+                                                        T_, C, act)
+#define BOTH(T)                        \
+  do {                                 \
+    if (taps == 2) VEC(T, 2);          \
+    else if (taps == 3) VEC(T, 3);     \
+    else VEC(T, 4);                    \
+    conv_state_kernel<T><<<g2, threads, 0, stream>>>((const T*)xin, in_stride, conv_state, row_slot, row_q_start, row_q_len, C, taps, in_bias); \
+  } while (0)
+    if (dtype == DK_F32) BOTH(float);
+    else BOTH(__nv_bfloat16);
+#undef BOTH
+#undef VEC
+    return dk_check_launch("conv_silu");
+  }
   if (dtype == DK_F32) {
     conv_silu_kernel<float><<<g1, threads, 0, stream>>>((const float*)xin, in_stride, w, bias, conv_state, (float*)out, tok_row,
                                                         row_slot, row_q_start, C, taps, in_bias, act);

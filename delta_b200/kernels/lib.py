@@ -54,7 +54,7 @@ _SIGNATURES = {
     "dk_stream_norm": [P, P, P, P, P, P, P, P, I, I, I, F, I, I, I, P],
     "dk_activation": [P, P, L, I, I, P],
     "dk_softcap": [P, L, F, F, P],
-    "dk_conv_silu": [P, I, P, P, P, P, P, P, P, P, I, I, I, I, P, I, I, P],
+    "dk_conv_silu": [P, I, P, P, P, P, P, P, P, P, I, I, I, I, P, I, I, I, P],
     "dk_selective_scan": [P, P, P, I, I, I, P, I, P, P, P, P, P, P, P, P, I, I, I, I, I, I, P, P, P],
     "dk_attention_rows_plain": [C.POINTER(RowAttnParams), P],
     "dk_rows_append": [P, I, P, P, P, I, P, I, P, I, I, I, I, I, I, I, I, I, I, I, I, I, P, P],
@@ -89,9 +89,9 @@ _SIGNATURES = {
     "dk_gemm_stream_k_supported": [I, I, I, I],
     "dk_gemm_stream_k": [P, P, P, I, I, I, I, I, I, I, I, P, P, P],
     "dk_wait_check": [P, C.c_longlong, P],
-    "dk_embedding_pair": [P, P, P, P, P, P, P, F, P, L, L, L, P, P, P, I, I, I, I, P, P],
+    "dk_embedding_pair": [P, P, P, P, P, P, P, F, P, L, L, L, P, P, P, P, P, F, I, I, I, I, I, P, P],
     "dk_remember_tokens": [P, P, P, P, P, I, P],
-    "dk_residual_norm": [P, P, P, P, P, P, P, P, P, I, I, F, I, I, I, I, P],
+    "dk_residual_norm": [P, P, P, F, P, P, P, P, P, P, I, I, F, I, I, I, I, P],
     "dk_sublayer_norm_add": [P, P, P, P, P, I, I, F, I, I, I, P],
     "dk_rows_append_unit": [P, I, P, P, P, I, P, I, P, I, I, I, I, I, I, I, I, I, I, I, I, I, F, I, P, P, P, F, I, F, I, I, P, P],
     "dk_decay_attention_slice": [I, I, I, I],
@@ -112,16 +112,28 @@ _SIGNATURES = {
     "dk_matrix_memory_chunk": [],
     "dk_matrix_memory_chunked_supported": [I, I],
     "dk_matrix_memory_chunked": [P, I, I, I, I, F, P, P, F, F, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P],
-    "dk_gated_rms_norm": [P, P, I, P, P, I, I, F, I, I, P],
+    "dk_gated_rms_norm": [P, P, I, P, P, I, I, F, I, I, I, I, P],
+    "dk_delta_rule_max_key": [],
+    "dk_delta_rule": [P, I, I, I, P, I, P, I, P, P, P, P, P, P, P, I, I, I, I, I, F, F, I, P],
+    "dk_delta_rule_chunk": [],
+    "dk_delta_rule_chunked_supported": [I, I],
+    "dk_delta_rule_chunk_floats": [I, I],
+    "dk_delta_rule_chunked": [P, I, I, I, P, I, P, I, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, F, I, P],
+    "dk_state_space_max_state": [],
+    "dk_state_space": [P, I, P, I, P, P, P, P, P, P, P, P, I, I, I, I, I, I, P],
+    "dk_state_space_chunk": [],
+    "dk_state_space_chunked_supported": [I, I],
+    "dk_state_space_chunk_floats": [I, I],
+    "dk_state_space_chunked": [P, I, P, I, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P],
     "dk_glu_clamped": [P, P, L, I, F, F, F, F, I, P],
     "dk_router_topk": [P, I, P, P, I, I, I, P],
-    "dk_router": [P, P, P, P, P, I, I, I, I, I, P, F, I, I, P],
+    "dk_router": [P, P, P, P, P, I, I, I, I, I, P, F, I, I, I, I, P],
     "dk_experts_align": [P, I, I, P, I, P, I, I, P],
     "dk_experts_gather": [P, P, I, P, I, I, P, P],
     "dk_experts_gemm_tc_supported": [I, I, I],
     "dk_experts_gemm_tc": [P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, F, P, P],
     "dk_experts_gemm": [P, P, P, P, P, I, I, I, I, I, F, F, F, P, I, P],
-    "dk_experts_combine": [P, P, I, P, P, I, P, I, I, I, P],
+    "dk_experts_combine": [P, P, I, P, P, I, P, I, I, P, P, I, I, I, P],
     "dk_experts_tile_rows": [],
 }
 

@@ -480,11 +480,13 @@ def softcap(logits, cap: Optional[float], scale: float = 1.0):
 
 # ---- the selective state-space mixer ----------------------------------------------------------------------
 
-def conv_silu(xin, in_stride, weight, bias, conv_state, out, *, tok_row, row_slot, row_q_start, row_q_len, in_bias=None, silu=True):
+def conv_silu(xin, in_stride, weight, bias, conv_state, out, *, tok_row, row_slot, row_q_start, row_q_len, in_bias=None, silu=True,
+              single=False):
     """Causal convolution over each row's tokens and silu; ``xin`` holds a token's C inputs at the start of rows of
     ``in_stride`` elements.  ``conv_state`` [slots, taps-1, C] (float32) supplies the inputs before the step's first
     token and is left holding the last taps-1 inputs of every row.  ``in_bias`` (float32 [C]) is added to every input
-    as it is read (the zeros before a request's first token stay zeros); ``silu`` False: no activation."""
+    as it is read (the zeros before a request's first token stay zeros); ``silu`` False: no activation.  ``single``: every row
+    brings one token (one kernel does both)."""
     T, C_ = out.shape
     taps = weight.shape[1]
     i32, f32 = torch.int32, torch.float32
@@ -492,7 +494,8 @@ def conv_silu(xin, in_stride, weight, bias, conv_state, out, *, tok_row, row_slo
         _ptr(xin, "xin", out.dtype), int(in_stride), _ptr(weight, "weight", f32), _ptr(bias, "bias", f32),
         _ptr(conv_state, "conv_state", f32), _ptr(out, "out"), _ptr(tok_row, "tok_row", i32), _ptr(row_slot, "row_slot", i32),
         _ptr(row_q_start, "row_q_start", i32), _ptr(row_q_len, "row_q_len", i32), T, row_slot.shape[0], C_, taps,
-        _ptr(in_bias, "in_bias", f32), int(bool(silu)), dtype_code(out.dtype), _stream()), "conv_silu", 2 if taps > 1 else 1)
+        _ptr(in_bias, "in_bias", f32), int(bool(silu)), int(bool(single)), dtype_code(out.dtype), _stream()), "conv_silu",
+        2 if taps > 1 and not single else 1)
     return out
 
 
@@ -655,17 +658,20 @@ NORM_KINDS = {"rms": 0, "layer": 1}
 
 
 def embedding_pair(tokens, table, X, *, scale=1.0, pair_table=None, buckets=0, mul_prev=0, mul_cur=0, prev_state=None, tok_row=None,
-                   tok_pos=None, row_q_start=None, row_slot=None, keep=None, rounded=None, err=None):
+                   tok_pos=None, row_q_start=None, row_slot=None, keep=None, rounded=None, norm_weight=None, norm_bias=None, eps=0.0, kind="rms",
+                   err=None):
     """X[t] = table[tokens[t]] * scale (+ pair_table[(previous token * mul_prev + token * mul_cur) mod buckets]; a request's
     first token takes row ``buckets``; the token before a portion's first comes from ``prev_state`` [slots, 1]).  X, and
-    ``keep`` when given (a second copy), are float32 [T, d]; ``rounded`` when given takes X in the table's type."""
+    ``keep`` when given (a second copy), are float32 [T, d]; ``rounded`` when given takes X in the table's type.
+    ``norm_weight`` (float32 [d]): X is normed over the width first (``kind`` "rms" or "layer"), times the weight, plus ``norm_bias``."""
     T, d = X.shape
     i32 = torch.int32
     _l.check(_l.load().dk_embedding_pair(
         _ptr(tokens, "tokens", i32), _ptr(tok_row, "tok_row", i32), _ptr(tok_pos, "tok_pos", i32), _ptr(row_q_start, "row_q_start", i32),
         _ptr(row_slot, "row_slot", i32), _ptr(prev_state, "prev_state", i32), _ptr(table, "table"), float(scale),
         _ptr(pair_table, "pair_table", table.dtype), int(buckets), int(mul_prev), int(mul_cur), _ptr(X, "X", torch.float32),
-        _ptr(keep, "keep", torch.float32), _ptr(rounded, "rounded", table.dtype), T, d, table.shape[0], dtype_code(table.dtype), _ptr(err, "err", i32), _stream()), "embedding_pair")
+        _ptr(keep, "keep", torch.float32), _ptr(rounded, "rounded", table.dtype), _ptr(norm_weight, "norm_weight", torch.float32),
+        _ptr(norm_bias, "norm_bias", torch.float32), float(eps), NORM_KINDS[kind], T, d, table.shape[0], dtype_code(table.dtype), _ptr(err, "err", i32), _stream()), "embedding_pair")
     return X
 
 
@@ -677,8 +683,9 @@ def remember_tokens(tokens, prev_state, *, row_q_start, row_q_len, row_slot):
              "remember_tokens")
 
 
-def residual_norm(X, out, *, updates=(), extra=None, vec=None, weight=None, bias=None, eps=0.0, kind="layer", rows=None, write_back=True):
-    """The step between two layers on a 32-bit stream X [T, d]:  X <- X + (y1 + y2) (``updates``: none, one or two tensors
+def residual_norm(X, out, *, updates=(), update_scale=1.0, extra=None, vec=None, weight=None, bias=None, eps=0.0, kind="layer", rows=None,
+                  write_back=True):
+    """The step between two layers on a 32-bit stream X [T, d]:  X <- X + ``update_scale`` (y1 + y2) (``updates``: none, one or two tensors
     of the compute type), X <- X + ``extra`` (float32 [T, d]), X <- X + ``vec`` (float32 [d]), stored when ``write_back``;
     then ``out`` = norm(X) * weight with the layer norm without bias or the RMS norm (``weight`` None: X itself).
     ``bias`` (float32 [d]) is added behind the weight.  ``rows``: only these tokens, in this order.  ``out`` None: only the sums
@@ -697,7 +704,7 @@ def residual_norm(X, out, *, updates=(), extra=None, vec=None, weight=None, bias
     f32 = torch.float32
     ydt = dtype_code(y1.dtype) if y1 is not None else (dtype_code(out.dtype) if out is not None and out.dtype != f32 else F32)
     _l.check(_l.load().dk_residual_norm(
-        _ptr(X, "X", f32), _ptr(y1, "update"), _ptr(y2, "update", y1.dtype if y1 is not None else None), _ptr(extra, "extra", f32),
+        _ptr(X, "X", f32), _ptr(y1, "update"), _ptr(y2, "update", y1.dtype if y1 is not None else None), float(update_scale), _ptr(extra, "extra", f32),
         _ptr(vec, "vec", f32), _ptr(weight, "weight", f32), _ptr(bias, "bias", f32) if weight is not None else None, _ptr(out, "out"),
         _ptr(rows, "rows", torch.int32), n, d, float(eps),
         NORM_KINDS[kind], int(bool(write_back)), ydt, dtype_code(out.dtype) if out is not None else F32, _stream()), "residual_norm")
@@ -786,13 +793,15 @@ def decay_attention_chunked(src, q_off, k_off, v_off, decays, state, out, work, 
     return out
 
 
-def gated_rms_norm(o, gate_ptr, gate_stride, weight, out, eps, group=None):
+def gated_rms_norm(o, gate_ptr, gate_stride, weight, out, eps, group=None, gate_first=False, gate_dtype=None):
     """out = o / sqrt(mean(o^2) + eps) * weight * sigmoid(gate) per token; ``o`` float32 [T, n]; the gate's n values of a token
     lie at ``gate_ptr`` + t * ``gate_stride`` elements of the type of ``out``.  ``group``: the mean is taken over every ``group``
-    consecutive entries (one head) instead of the whole row."""
+    consecutive entries (one head) instead of the whole row.  ``gate_first``: the gate multiplies before the norm, and through silu,
+    out = rms(o * silu(gate)) * weight.  ``gate_dtype``: the gate's type where it is not that of ``out``."""
     T, n = o.shape
     _l.check(_l.load().dk_gated_rms_norm(_ptr(o, "o", torch.float32), gate_ptr, int(gate_stride), _ptr(weight, "weight", torch.float32),
-                                         _ptr(out, "out"), T, n, float(eps), int(group or n), dtype_code(out.dtype), _stream()), "gated_rms_norm")
+                                         _ptr(out, "out"), T, n, float(eps), int(group or n), int(bool(gate_first)),
+                                         dtype_code(gate_dtype or out.dtype), dtype_code(out.dtype), _stream()), "gated_rms_norm")
     return out
 
 
@@ -941,6 +950,108 @@ def matrix_memory_chunked(src, q_off, k_off, v_off, q_scale, gates, gate_bias, c
     return out
 
 
+# ---- the gated delta rule --------------------------------------------------------------------------------------------
+
+def delta_rule_max_key() -> int:
+    return int(_l.load().dk_delta_rule_max_key())
+
+
+def delta_rule(qkv, k_off, v_off, b_ptr, b_stride, a, A_log, dt_bias, state, out, *, H, G, dk, dv, q_scale, guard, row_slot, row_q_start,
+               row_q_len=None):
+    """The gated delta rule with a decay per head and key channel over each row's tokens, from and into ``state``
+    [slots, H, dv, dk] (float32); ``csrc/delta_rule.cu`` has the equations.  ``qkv`` [T, stride] holds q (G heads of dk), k at ``k_off``
+    and v (H heads of dv) at ``v_off``, behind the convolution and before the unit norms; ``b_ptr`` points at a token's H values before
+    the sigmoid (rows of ``b_stride`` elements of qkv's type); ``a`` float32 [T, >= H*dk] the decays' raw values; ``out`` float32
+    [T, H*dv].  ``row_q_len`` None: every row brings one token."""
+    _check_shape(state, (H, dv, dk), "delta_rule")
+    i32, f32 = torch.int32, torch.float32
+    _l.check(_l.load().dk_delta_rule(
+        _ptr(qkv, "qkv"), qkv.shape[1], int(k_off), int(v_off), b_ptr, int(b_stride), _ptr(a, "a", f32), a.shape[1], _ptr(A_log, "A_log", f32),
+        _ptr(dt_bias, "dt_bias", f32), _ptr(state, "state", f32), _ptr(out, "out", f32), _ptr(row_slot, "row_slot", i32),
+        _ptr(row_q_start, "row_q_start", i32), _ptr(row_q_len, "row_q_len", i32), row_slot.shape[0], H, G, dk, dv, float(q_scale),
+        float(guard), dtype_code(qkv.dtype), _stream()), "delta_rule")
+    return out
+
+
+def delta_rule_chunk() -> int:
+    return int(_l.load().dk_delta_rule_chunk())
+
+
+def delta_rule_chunked_supported(dk, dv) -> bool:
+    return bool(_l.load().dk_delta_rule_chunked_supported(int(dk), int(dv)))
+
+
+def delta_rule_chunk_floats(dk, dv) -> int:
+    return int(_l.load().dk_delta_rule_chunk_floats(int(dk), int(dv)))
+
+
+def delta_rule_chunked(qkv, k_off, v_off, b_ptr, b_stride, a, A_log, dt_bias, state, out, work, chunk_base, max_chunks, *, H, G, dk, dv,
+                       q_scale, guard, row_slot, row_q_start, row_q_len):
+    """``delta_rule`` for long portions (two kernels: every chunk alone, then the states along each row).  ``chunk_base`` [rows] int32:
+    the chunks of all rows before each row; ``max_chunks``: the most chunks of a row; ``work`` float32 with
+    (all chunks) * H * ``delta_rule_chunk_floats`` entries."""
+    _check_shape(state, (H, dv, dk), "delta_rule_chunked")
+    i32, f32 = torch.int32, torch.float32
+    _l.check(_l.load().dk_delta_rule_chunked(
+        _ptr(qkv, "qkv"), qkv.shape[1], int(k_off), int(v_off), b_ptr, int(b_stride), _ptr(a, "a", f32), a.shape[1], _ptr(A_log, "A_log", f32),
+        _ptr(dt_bias, "dt_bias", f32), _ptr(state, "state", f32), _ptr(out, "out", f32), _ptr(work, "work", f32),
+        _ptr(row_slot, "row_slot", i32), _ptr(row_q_start, "row_q_start", i32), _ptr(row_q_len, "row_q_len", i32),
+        _ptr(chunk_base, "chunk_base", i32), row_slot.shape[0], int(max_chunks), H, G, dk, dv, float(q_scale), float(guard),
+        dtype_code(qkv.dtype), _stream()), "delta_rule_chunked", 2)
+    return out
+
+
+# ---- the state-space recurrence with one decay per head --------------------------------------------------------------
+
+def state_space_max_state() -> int:
+    return int(_l.load().dk_state_space_max_state())
+
+
+def state_space(xbc, dt_ptr, dt_stride, A_log, dt_bias, D, state, out, *, H, G, N, P, row_slot, row_q_start, row_q_len=None):
+    """The state-space recurrence with one decay per head over each row's tokens, from and into ``state`` [slots, H, P, N] (float32);
+    ``csrc/state_space.cu`` has the equations.  ``xbc`` [T, stride]: x (H heads of P), B and C (G groups of N) behind the convolution;
+    ``dt_ptr`` points at a token's H step sizes before bias and softplus (rows of ``dt_stride`` elements of xbc's type); ``out`` float32
+    [T, H*P].  ``row_q_len`` None: every row brings one token."""
+    _check_shape(state, (H, P, N), "state_space")
+    i32, f32 = torch.int32, torch.float32
+    _l.check(_l.load().dk_state_space(
+        _ptr(xbc, "xbc"), xbc.shape[1], dt_ptr, int(dt_stride), _ptr(A_log, "A_log", f32), _ptr(dt_bias, "dt_bias", f32), _ptr(D, "D", f32),
+        _ptr(state, "state", f32), _ptr(out, "out", f32), _ptr(row_slot, "row_slot", i32), _ptr(row_q_start, "row_q_start", i32),
+        _ptr(row_q_len, "row_q_len", i32), row_slot.shape[0], H, G, N, P, dtype_code(xbc.dtype), _stream()), "state_space")
+    return out
+
+
+def state_space_chunk() -> int:
+    return int(_l.load().dk_state_space_chunk())
+
+
+def state_space_chunked_supported(N, P) -> bool:
+    return bool(_l.load().dk_state_space_chunked_supported(int(N), int(P)))
+
+
+def state_space_chunk_floats(H, G) -> int:
+    return int(_l.load().dk_state_space_chunk_floats(int(H), int(G)))
+
+
+def state_space_chunked(xbc, dt_ptr, dt_stride, A_log, dt_bias, D, state, out, work, chunk_base, total_chunks, max_chunks, *, H, G, N, P,
+                        row_slot, row_q_start, row_q_len):
+    """``state_space`` for long portions (two kernels: every chunk's products and decays, then the states along each row).
+    ``work`` float32 with total_chunks * ``state_space_chunk_floats`` entries; the rest as for ``delta_rule_chunked``."""
+    _check_shape(state, (H, P, N), "state_space_chunked")
+    i32, f32 = torch.int32, torch.float32
+    _l.check(_l.load().dk_state_space_chunked(
+        _ptr(xbc, "xbc"), xbc.shape[1], dt_ptr, int(dt_stride), _ptr(A_log, "A_log", f32), _ptr(dt_bias, "dt_bias", f32), _ptr(D, "D", f32),
+        _ptr(state, "state", f32), _ptr(out, "out", f32), _ptr(work, "work", f32), _ptr(row_slot, "row_slot", i32),
+        _ptr(row_q_start, "row_q_start", i32), _ptr(row_q_len, "row_q_len", i32), _ptr(chunk_base, "chunk_base", i32), row_slot.shape[0],
+        int(total_chunks), int(max_chunks), H, G, N, P, dtype_code(xbc.dtype), _stream()), "state_space_chunked", 2)
+    return out
+
+
+def _check_shape(state, per_slot, who):
+    if tuple(state.shape[1:]) != tuple(per_slot):
+        raise KernelError(f"{who}: the state has shape {tuple(state.shape)}, expected [slots, {', '.join(str(n) for n in per_slot)}]")
+
+
 # ---- gated feed-forwards and a mixture of experts ---------------------------------------------------------------
 
 def glu_clamped(gate_up, out, limit=-1.0, alpha=1.702, shift=1.0, cubic=0.0):
@@ -959,18 +1070,24 @@ def router_topk(logits, experts, top, choice, weight):
                                       _ptr(weight, "weight", torch.float32), T, int(experts), int(top), _stream()), "router_topk")
 
 
-def router(x, w, experts, top, logits, choice, weight, scoring="softmax", correction=None, scale=1.0, normalize=True):
+ROUTER_SCORINGS = {"softmax": 0, "sigmoid": 1, "softmax_all": 3}
+
+
+def router(x, w, experts, top, logits, choice, weight, scoring="softmax", correction=None, scale=1.0, normalize=True, groups=None):
     """logits = x w^T in 32 bit ([T, rows of w]; the first ``experts`` rows are the experts'), and per token the ``top`` largest of
     the experts' logits with the softmax over them.  ``scoring`` "sigmoid": scores s = sigmoid(logit); the ``top`` largest of
     s + ``correction`` (float32 [experts] or None) are chosen; the weights are the chosen s divided by their sum (``normalize``
-    False: the chosen s themselves), times ``scale``."""
+    False: the chosen s themselves), times ``scale``.  ``scoring`` "softmax_all": the same with s the softmax over all ``experts`` logits.
+    ``groups`` (count, keep): the experts form that many equal groups of neighbours, and only those of the ``keep`` groups with the
+    largest s + correction in them can be chosen."""
     T, d = x.shape
-    if scoring not in ("softmax", "sigmoid"):
+    if scoring not in ROUTER_SCORINGS:
         raise KernelError(f"router: unknown scoring '{scoring}'")
     _l.check(_l.load().dk_router(_ptr(x, "x"), _ptr(w, "w", x.dtype), _ptr(logits, "logits", torch.float32), _ptr(choice, "choice", torch.int32),
                                  _ptr(weight, "weight", torch.float32), T, d, w.shape[0], int(experts), int(top),
                                  _ptr(correction, "correction", torch.float32), float(scale),
-                                 (1 if normalize else 2) if scoring == "sigmoid" else 0,
+                                 ROUTER_SCORINGS[scoring] + (0 if normalize or scoring == "softmax" else 1), int(groups[0]) if groups else 0,
+                                 int(groups[1]) if groups else 0,
                                  dtype_code(x.dtype), _stream()), "router")
 
 
@@ -1032,12 +1149,15 @@ def experts_gemm(a, w, out, sorted_slots, tile_expert, *, top, n, k, act=False, 
                                        dtype_code(a.dtype), _stream()), "experts_gemm")
 
 
-def experts_combine(z, weight, out, shared=None, gate_logit=None, gate_stride=0, top=None):
+def experts_combine(z, weight, out, shared=None, gate_logit=None, gate_stride=0, top=None, identity=None):
     """out[t] = sum_j weight[t, j] z[t*top + j] (+ sigmoid(gate logit of t) * shared[t]; no gate logit: + shared[t]); ``gate_logit``: an
-    address (float32).  ``weight`` None with ``top``: every weight is 1."""
+    address (float32).  ``weight`` None with ``top``: every weight is 1.  ``identity`` (x, choice, first): a choice from ``first`` on adds
+    weight * x[t] instead of a row of z."""
     T, d = out.shape
+    x, choice, first = identity or (None, None, 0)
     _l.check(_l.load().dk_experts_combine(_ptr(z, "z", torch.float32), _ptr(weight, "weight", torch.float32),
                                           weight.shape[1] if weight is not None else int(top),
-                                          _ptr(shared, "shared", out.dtype), gate_logit, int(gate_stride), _ptr(out, "out"), T, d,
+                                          _ptr(shared, "shared", out.dtype), gate_logit, int(gate_stride), _ptr(out, "out"), T, d, _ptr(x, "x"),
+                                          _ptr(choice, "choice", torch.int32), int(first), dtype_code(x.dtype if x is not None else out.dtype),
                                           dtype_code(out.dtype), _stream()), "experts_combine")
     return out

@@ -24,7 +24,7 @@ class Model:
         self.spec = spec
         self.blocks = []
         for ls in spec.layers:
-            self.blocks.append(BLOCKS.create(ls.block, parts={role: ps.build() for role, ps in ls.parts.items()}))
+            self.blocks.append(BLOCKS.create(ls.block, parts={role: ps.build() for role, ps in ls.parts.items()}, **ls.options))
         self.final_norm = spec.final_norm.build(NORMS)
         self.stream = spec.stream.build(STREAMS) if spec.stream is not None else STREAMS.create("single", width=spec.width)
         self.embed_table = None

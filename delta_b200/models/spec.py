@@ -11,9 +11,11 @@ from ..parts.base import PartSpec, TensorSpec
 class LayerSpec:
     """One layer: a block arrangement and the parts it is built from, by the role each
     plays in that block (the pre-norm block: norm1, mixer, norm2, feed_forward).  Every
-    ``PartSpec`` names its registry in ``category``."""
+    ``PartSpec`` names its registry in ``category``.  ``options`` are constants of the
+    arrangement itself (what a block takes beside its parts)."""
     parts: Mapping[str, PartSpec]
     block: str = "pre_norm"
+    options: Mapping = field(default_factory=dict)
 
 
 @dataclass(frozen=True)

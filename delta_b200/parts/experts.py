@@ -11,7 +11,10 @@ rows of one expert, and the two products of all experts are one launch each: war
 by side (``csrc/gemm_tc.cu``).  The router's rows and
 the shared expert's gate row are one matrix, so one product gives both.
 
-Options: ``scoring`` "sigmoid": scores s = sigmoid(z); the ``top`` largest of s + correction (a tensor ``correction`` [E] when
+Options: ``scoring`` "softmax_all": as "sigmoid" below with s = the softmax over all of the router's logits.  ``groups`` (count, keep): the
+router's outputs form that many equal groups of neighbours; a group's score is the largest s + correction in it, and only outputs of the
+``keep`` best groups can be chosen.  ``identity`` n: the router has n more outputs than there are experts, the last ones; a token that
+chooses one of them gets its own input h times the weight (no tensors, no product).  ``scoring`` "sigmoid": scores s = sigmoid(z); the ``top`` largest of s + correction (a tensor ``correction`` [E] when
 ``correction`` is set) are chosen, and the weights are the chosen s (without the correction) divided by their sum (+ 1e-20), times
 ``route_scale``; ``normalize`` False: the chosen s themselves, times ``route_scale``.  ``weight_input``: a choice's weight multiplies
 what its expert reads, out = sum expert(weight * h), not what it gives: since (w h) W^T = w (h W^T), the first product's result is
@@ -42,28 +45,35 @@ class Experts(FeedForward):
     def __init__(self, prefix: str, width: int, experts: int, top: int, intermediate: int, limit=None, alpha: float = 1.702,
                  shift: float = 1.0, shared: Optional[dict] = None, scoring: str = "softmax", correction: bool = False,
                  route_scale: float = 1.0, activation: str = "clamped_glu", wide_output: bool = False, normalize: bool = True,
-                 weight_input: bool = False):
+                 weight_input: bool = False, identity: int = 0, groups: Optional[tuple] = None):
         self.prefix, self.width = prefix, int(width)
         self.experts, self.top, self.intermediate = int(experts), int(top), int(intermediate)
-        if not (1 <= self.top <= self.experts):
+        self.identity, self.outputs = int(identity), int(experts) + int(identity)      # the router's outputs: experts, then identities
+        self.groups = (int(groups[0]), int(groups[1])) if groups else None
+        if not (1 <= self.top <= self.outputs):
             raise ValueError(f"{self.top} of {self.experts} experts cannot be chosen")
         if limit is not None and float(limit) < 0:
             raise ValueError(f"a clamp at {limit} is no limit")
         self.limit, self.alpha, self.shift = (-1.0 if limit is None else float(limit)), float(alpha), float(shift)
-        if scoring not in ("softmax", "sigmoid"):
-            raise ValueError(f"unknown router scoring '{scoring}' (softmax, sigmoid)")
+        if scoring not in ops.ROUTER_SCORINGS:
+            raise ValueError(f"unknown router scoring '{scoring}' ({', '.join(ops.ROUTER_SCORINGS)})")
+        if self.groups and (scoring == "softmax" or self.outputs % self.groups[0] or not 1 <= self.groups[1] <= self.groups[0]
+                            or self.groups[1] * (self.outputs // self.groups[0]) < self.top):
+            raise ValueError(f"{self.groups[1]} of {self.groups[0]} groups of {self.outputs} experts do not hold {self.top} choices")
+        if self.identity and (shared or weight_input):
+            raise ValueError("identity experts beside a shared expert, or with weights on the experts' inputs, are not built")
         if activation not in ("clamped_glu", "relu_squared"):
             raise ValueError(f"unknown expert activation '{activation}' (clamped_glu, relu_squared)")
-        if correction and scoring != "sigmoid":
-            raise ValueError("a correction of the choice belongs to sigmoid scores")
+        if correction and scoring == "softmax":
+            raise ValueError("a correction of the choice belongs to scores (sigmoid, softmax_all)")
         self.scoring, self.has_correction, self.route_scale = scoring, bool(correction), float(route_scale)
         self.gated = activation == "clamped_glu"
         self.wide_output = bool(wide_output)
         if self.wide_output and shared:
             raise ValueError("the 32-bit output is for experts without a shared expert (whose output has the compute type)")
         self.normalize, self.weight_input = bool(normalize), bool(weight_input)
-        if not self.normalize and scoring != "sigmoid":
-            raise ValueError("weights that are not normalised belong to sigmoid scores")
+        if not self.normalize and scoring == "softmax":
+            raise ValueError("weights that are not normalised belong to scores (sigmoid, softmax_all)")
         self.correction = None
         self.shared = None
         self.shared_gate = bool(shared.get("gate", True)) if shared else False
@@ -74,9 +84,9 @@ class Experts(FeedForward):
 
     def tensor_specs(self):
         p, d, F = self.prefix, self.width, self.intermediate
-        specs = [TensorSpec(p + "router", (self.experts, d))]
+        specs = [TensorSpec(p + "router", (self.outputs, d))]
         if self.has_correction:
-            specs.append(TensorSpec(p + "correction", (self.experts,), kind="vector", init="uniform:-0.2:0.2"))
+            specs.append(TensorSpec(p + "correction", (self.outputs,), kind="vector", init="uniform:-0.2:0.2"))
         for e in range(self.experts):
             specs += ([TensorSpec(f"{p}e{e}.gate", (F, d))] if self.gated else []) + [TensorSpec(f"{p}e{e}.up", (F, d)),
                                                                                      TensorSpec(f"{p}e{e}.down", (d, F))]
@@ -103,8 +113,8 @@ class Experts(FeedForward):
         z = torch.empty((T, self.w_router.shape[0]), dtype=f32, device=dev)        # [T, E (+1)]
         choice = torch.empty((T, top), dtype=i32, device=dev)
         weight = torch.empty((T, top), dtype=f32, device=dev)
-        ops.router(x, self.w_router, E, top, z, choice, weight, scoring=self.scoring, correction=self.correction, scale=self.route_scale,
-                   normalize=self.normalize)
+        ops.router(x, self.w_router, self.outputs, top, z, choice, weight, scoring=self.scoring, correction=self.correction, scale=self.route_scale,
+                   normalize=self.normalize, groups=self.groups)
         act = "gated" if self.gated else "relu_squared"
         slots = T * top
         # weight_input: a slot's weight goes into the first product (or into the gathered rows), and the sum at the end has none
@@ -133,8 +143,8 @@ class Experts(FeedForward):
             weight = None
         if self.shared is not None:
             s = self.shared.forward(ctx, x)
-            ops.experts_combine(out_slots, weight, out, shared=s, gate_logit=(z.data_ptr() + E * 4) if self.shared_gate else None,
+            ops.experts_combine(out_slots, weight, out, shared=s, gate_logit=(z.data_ptr() + self.outputs * 4) if self.shared_gate else None,
                                 gate_stride=z.shape[1], top=top)
-        else:
-            ops.experts_combine(out_slots, weight, out, top=top)
+        else:      # a choice behind the experts' numbers is left out of the sorted tiles; the sum takes the input for it
+            ops.experts_combine(out_slots, weight, out, top=top, identity=(x, choice, E) if self.identity else None)
         return out

@@ -11,6 +11,9 @@ value size ``value_dim``, latent size R):
     s_h(i, j)    = (q_h^plain(i) . k_h^plain(j) + rot(q_h^rot(i)) . r(j)) * scale ,  causal softmax over j <= i
 With ``q_rank`` Rq the queries go through a latent of their own, c_q = rmsnorm(W_dq h) * w_q, q = W_uq c_q (tensors ``dq``, ``dq.norm``,
 ``uq`` instead of ``q``): W_dq rides with W_dkv in the first product, and a second product makes the heads' queries.
+Options: ``window`` W, query i sees the keys j with i - W < j <= i (None: every j <= i); ``sink``, a learned logit per head that joins
+the softmax's denominator and carries no value; ``gate``, the heads' outputs are multiplied by sigmoid(W_g h) before the output
+projection (W_g's rows ride in the first product).
 The keys are never made: since q^plain . (U^K c) = ((U^K)^T q^plain) . c, the query is carried into the latent
 space once per new token (one product per head), attention then runs with one shared key-value head whose key is the
 cached row [c | r] and whose value is c, and U^V is applied to the attended latent afterwards.  So a step's cost
@@ -55,12 +58,14 @@ def heads_product(ctx, a, a_off, lda, sa, w, n, k, c, c_off, ldc, sc, heads):
 class LatentAttention(Mixer):
     """Tensor names under ``prefix``: ``q`` [H*(head_dim+rot_dim), d] (with ``q_rank`` Rq instead ``dq`` [Rq, d], ``dq.norm`` [Rq],
     ``uq`` [H*(head_dim+rot_dim), Rq]), ``dkv`` [R+rot_dim, d], ``dkv.norm`` [R], ``uk`` [H*head_dim, R], ``uv`` [H*value_dim, R],
-    ``o`` [d, H*value_dim]."""
+    ``o`` [d, H*value_dim]; with the options ``sink`` [H], ``g`` [H*value_dim, d]."""
 
     def __init__(self, prefix: str, width: int, heads: int, head_dim: int, rot_dim: int, value_dim: int, kv_rank: int,
                  eps: float, scale: Optional[float] = None, position: Optional[PartSpec] = None, rot_dims: Optional[int] = None,
-                 q_rank: Optional[int] = None):
+                 q_rank: Optional[int] = None, window: Optional[int] = None, sink: bool = False, gate: bool = False):
         self.q_rank = int(q_rank) if q_rank else 0
+        self.window, self.has_sink, self.has_gate = (int(window) if window else None), bool(sink), bool(gate)
+        self.sink = None
         self.w_uq = self.q_norm_w = None
         self.prefix, self.width = prefix, int(width)
         self.heads, self.dq, self.dr, self.dv, self.rank = int(heads), int(head_dim), int(rot_dim), int(value_dim), int(kv_rank)
@@ -79,15 +84,24 @@ class LatentAttention(Mixer):
                        TensorSpec(p + "uq", (H * (self.dq + self.dr), self.q_rank))]
         else:
             queries = [TensorSpec(p + "q", (H * (self.dq + self.dr), d))]
+        options = [TensorSpec(p + "sink", (H,), kind="vector", init="uniform:-1:1")] if self.has_sink else []
+        options += [TensorSpec(p + "g", (H * self.dv, d))] if self.has_gate else []
         return queries + [TensorSpec(p + "dkv", (self.rank + self.dr, d)),
                 TensorSpec(p + "dkv.norm", (self.rank,), kind="vector", init="norm"),
                 TensorSpec(p + "uk", (H * self.dq, self.rank)), TensorSpec(p + "uv", (H * self.dv, self.rank)),
-                TensorSpec(p + "o", (d, H * self.dv))]
+                TensorSpec(p + "o", (d, H * self.dv))] + options
 
     def bind(self, tensors):
         p, H = self.prefix, self.heads
         first = tensors[p + "dq"] if self.q_rank else tensors[p + "q"]
-        self.w_in = torch.cat([first, tensors[p + "dkv"]], dim=0).contiguous()      # one product for q (or its latent) and the latent
+        rows = [first, tensors[p + "dkv"]]      # one product for q (or its latent), the latent, and the output gate
+        if self.has_gate:
+            used = sum(t.shape[0] for t in rows)
+            if used % 8:      # the gate begins on a 16-byte boundary
+                rows.append(first.new_zeros((-used % 8, self.width)))
+            rows.append(tensors[p + "g"])
+        self.w_in = linear.padded_rows(torch.cat(rows, dim=0)) if self.has_gate else torch.cat(rows, dim=0).contiguous()
+        self.sink = tensors[p + "sink"].float().contiguous() if self.has_sink else None
         if self.q_rank:
             self.w_uq = tensors[p + "uq"]
             self.q_norm_w = tensors[p + "dq.norm"]
@@ -98,13 +112,14 @@ class LatentAttention(Mixer):
 
     def cache_spec(self):
         # a page of a layer: [one shared head][offset in the page][latent | rotated key part]
-        return CacheSpec((1, PAGE, self.rank + self.dr), None, run_tokens=128)
+        return CacheSpec((1, PAGE, self.rank + self.dr), self.window, run_tokens=128)
 
     def forward(self, ctx, x, cache):
         H, dq, dr, dv, R = self.heads, self.dq, self.dr, self.dv, self.rank
         T = x.shape[0]
         width = R + dr
-        src = linear.linear(ctx, x, self.w_in)                       # [T, H*(dq+dr) + R + dr], or [T, Rq + R + dr]
+        src = linear.linear(ctx, x, self.w_in)                       # [T, H*(dq+dr) + R + dr], or [T, Rq + R + dr] (and the gate)
+        first = src
         low, low_offset = None, 0
         if self.q_rank:
             cq = torch.empty((T, self.q_rank), dtype=x.dtype, device=x.device)
@@ -121,8 +136,12 @@ class LatentAttention(Mixer):
         heads_product(ctx, src, 0, src.shape[1], dq + dr, self.w_ukT, R, dq, qabs, 0, H * width, width, H)
         lat = torch.empty((T, H * R), dtype=x.dtype, device=x.device)
         params = row_attention.make_params(ctx, q=qabs, q_stride=H * width, q_head_stride=width, out=lat, cache=cache, H=H, KV=1,
-                                           dk=width, dv=R, row_width=width, k_off=0, v_off=0, scale=self.scale)
+                                           dk=width, dv=R, row_width=width, k_off=0, v_off=0, scale=self.scale,
+                                           window=self.window, sink=self.sink)
         row_attention.run(ctx, params)
         vals = torch.empty((T, H * dv), dtype=x.dtype, device=x.device)
         heads_product(ctx, lat, 0, H * R, R, self.w_uv, dv, R, vals, 0, H * dv, dv, H)
+        if self.has_gate:
+            at = (self.q_rank or H * (dq + dr)) + width
+            ops.sigmoid_gate(vals, first.data_ptr() + (at + -at % 8) * first.element_size(), first.shape[1], vals)
         return linear.linear(ctx, vals, self.w_o)

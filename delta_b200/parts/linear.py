@@ -240,6 +240,13 @@ def linear(ctx, x: torch.Tensor, w: torch.Tensor, out_dtype=None) -> torch.Tenso
     return out
 
 
+def padded_rows(w: torch.Tensor, multiple: int = 8) -> torch.Tensor:
+    """w with zero rows behind it up to a multiple of ``multiple``, so that the product's rows begin on 16-byte boundaries
+    (whoever reads them leaves the last columns alone)."""
+    short = -w.shape[0] % multiple
+    return torch.cat([w, w.new_zeros((short, w.shape[1]))], dim=0).contiguous() if short else w.contiguous()
+
+
 def linear_f32(ctx, x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     """x W^T with the sums left in 32 bit (for results that join a 32-bit stream or a recurrence unrounded)."""
     return linear(ctx, x, w, out_dtype=torch.float32)

@@ -13,36 +13,41 @@ from .base import NORMS, Norm, TensorSpec
 class RMSNorm(Norm):
     """``width`` and ``eps`` are parameters.  ``cast_before_weight`` keeps the order of
     the reference in reduced precision: the normalised value is rounded to the
-    activation type before it is multiplied by the weight (model.py:531-532)."""
+    activation type before it is multiplied by the weight (model.py:531-532).
+    ``weight_offset``: what is added to the stored weight, in 32 bit (1: the folder stores the
+    weight's deviation from one)."""
 
     kind = "rms"       # what a kernel that normalises a 32-bit stream is told
 
-    def __init__(self, name: str, width: int, eps: float, cast_before_weight: bool = True):
+    def __init__(self, name: str, width: int, eps: float, cast_before_weight: bool = True, weight_offset: float = 0.0):
         self.name = name
         self.width = int(width)
         self.eps = float(eps)
         self.cast_before_weight = bool(cast_before_weight)
+        self.weight_offset = float(weight_offset)
         self.weight = None
         self._weight32 = None
 
     def tensor_specs(self):
-        return [TensorSpec(self.name, (self.width,), kind="vector", init="norm")]
+        init = "norm" if not self.weight_offset else f"uniform:{0.9 - self.weight_offset}:{1.1 - self.weight_offset}"
+        return [TensorSpec(self.name, (self.width,), kind="vector", init=init)]
 
     def bind(self, tensors):
         self.weight = tensors[self.name]
         self._weight32 = None
 
     def weight32(self):
-        """The weight in 32 bit, for kernels that normalise a 32-bit stream."""
+        """The weight in 32 bit (with the offset), for kernels that normalise a 32-bit stream."""
         if self._weight32 is None:
-            self._weight32 = self.weight.float().contiguous()
+            self._weight32 = (self.weight.float() + self.weight_offset if self.weight_offset else self.weight.float()).contiguous()
         return self._weight32
 
     def forward(self, ctx, x, add=None, rows=None):
         n = x.shape[0] if rows is None else rows.shape[0]
         out = torch.empty((n, self.width), dtype=x.dtype, device=x.device)
         cast_first = self.cast_before_weight and x.dtype != torch.float32
-        return ops.rms_norm(x, self.weight, self.eps, out, add=add, rows=rows, cast_first=cast_first)
+        weight = self.weight32() if self.weight_offset else self.weight
+        return ops.rms_norm(x, weight, self.eps, out, add=add, rows=rows, cast_first=cast_first)
 
 
 @NORMS.register("layer_norm")

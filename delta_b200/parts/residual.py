@@ -3,9 +3,10 @@
 ``residual_f32``: x [T, d] float32.  It starts as
     x = table[token] * scale  (+ pair_table[(previous token * mul_prev + token * mul_cur) mod buckets])
 where the pair table ("bigram embedding") is optional; a request's first token takes the table's last row, and the
-token before a portion's first one is per-request state (``stream.prev_token``).  What a layer hands on as ``pending`` is
+token before a portion's first one is per-request state (``stream.prev_token``).  With ``start_norm`` the sum then goes through
+that norm, in 32 bit and in the same kernel.  What a layer hands on as ``pending`` is
 a ``Pending``: the outputs of its sublayers, not yet added, and what a re-entry adds.  The next norm adds them while it
-reads the stream (one kernel, ``ops.residual_norm``): x <- x + (y1 + y2), then + the embedding output, then + the pass's
+reads the stream (one kernel, ``ops.residual_norm``): x <- x + scale (y1 + y2) with the block's constant, then + the embedding output, then + the pass's
 vector.  ``reentry`` describes a span of layers that runs several times: before every pass but the first the embedding
 output (x as ``start`` made it) is added, and before every pass t the row t of the tensor ``reentry["name"]``
 [passes, d].
@@ -18,7 +19,8 @@ next norm adds, so the sum costs no kernel.
 ``parallel`` block: h = norm1(x); x <- x + (mixer(h) + feed_forward(h)); one norm, both sublayers read it; the
 feed-forward may be absent.
 
-``residual_pre_norm`` block: x <- x + mixer(norm1(x)); x <- x + feed_forward(norm2(x)); the second sublayer may be absent.
+``residual_pre_norm`` block: x <- x + m mixer(norm1(x)); x <- x + m feed_forward(norm2(x)) with a constant m (``update_scale``, 1
+unless given); the second sublayer may be absent.
 
 ``sublayer_norm`` block: the norms sit on the sublayers' outputs and the sublayers read the stream itself,
 x <- x + norm1(mixer(x)); x <- x + norm2(feed_forward(x)) (a norm may carry a scale per column behind it, "layer scale"); the second
@@ -34,7 +36,7 @@ import torch
 
 from ..kernels import ops
 from . import linear
-from .base import BLOCKS, STREAMS, Block, StateSpec, Stream, TensorSpec
+from .base import BLOCKS, NORMS, STREAMS, Block, PartSpec, StateSpec, Stream, TensorSpec
 
 PREV_TOKEN = "stream.prev_token"
 KEPT = "residual.embedding_output"
@@ -47,8 +49,13 @@ class Pending:
     updates: tuple = ()                       # outputs of the last layer's sublayers [T, d], compute type
     extra: Optional[torch.Tensor] = None      # float32 [T, d]
     vec: Optional[torch.Tensor] = None        # float32 [d]
+    scale: float = 1.0                        # the constant that multiplies the updates
     rounded: Optional[torch.Tensor] = None    # the settled stream in the compute type, when nothing above is pending and a kernel
                                               # made it on its way (a block whose sublayers read the stream itself takes it)
+
+    def sums(self) -> dict:
+        """What ``ops.residual_norm`` is to add."""
+        return dict(updates=self.updates, update_scale=self.scale, extra=self.extra, vec=self.vec)
 
     def empty(self) -> bool:
         return not self.updates and self.extra is None and self.vec is None
@@ -61,21 +68,21 @@ def read(ctx, x, pending: Optional[Pending], norm, rows=None, write_back=True):
     n = x.shape[0] if rows is None else rows.shape[0]
     if norm is None:
         out = torch.empty((n, x.shape[1]), dtype=torch.float32, device=x.device)
-        return ops.residual_norm(x, out, updates=p.updates, extra=p.extra, vec=p.vec, rows=rows, write_back=write_back)
+        return ops.residual_norm(x, out, **p.sums(), rows=rows, write_back=write_back)
     out = torch.empty((n, x.shape[1]), dtype=ctx.dtype, device=x.device)
     bias = norm.bias32() if hasattr(norm, "bias32") else None
-    return ops.residual_norm(x, out, updates=p.updates, extra=p.extra, vec=p.vec, weight=norm.weight32(), bias=bias, eps=norm.eps, kind=norm.kind,
-                             rows=rows, write_back=write_back)
+    return ops.residual_norm(x, out, **p.sums(), weight=norm.weight32(), bias=bias, eps=norm.eps, kind=norm.kind, rows=rows, write_back=write_back)
 
 
 @STREAMS.register("residual_f32")
 class ResidualStream(Stream):
     def __init__(self, width: int, scale: float = 1.0, pair: Optional[dict] = None, reentry: Optional[dict] = None,
-                 rounded_start: bool = False):
+                 rounded_start: bool = False, start_norm: Optional[PartSpec] = None):
         """``pair``: {name, buckets, mul_prev, mul_cur} of the hashed pair table [buckets + 1, d] (None: none).
         ``reentry``: {name, passes, add_embedding}, or {project, passes} (None: no span runs more than once).
         ``rounded_start``: the embedding kernel also leaves the stream in the compute type and ``initial_pending`` hands it to the
-        first block (for blocks whose sublayers read the stream itself)."""
+        first block (for blocks whose sublayers read the stream itself).  ``start_norm``: a norm that the embedding goes through."""
+        self.start_norm = start_norm.build(NORMS) if start_norm is not None else None
         self.rounded_start = bool(rounded_start)
         self._rounded = None
         self.width, self.scale = int(width), float(scale)
@@ -85,7 +92,7 @@ class ResidualStream(Stream):
         self.pair_table = self.pass_vectors = self.w_stream = self.w_embed = None
 
     def tensor_specs(self):
-        specs = []
+        specs = self.start_norm.tensor_specs() if self.start_norm is not None else []
         if self.pair:
             specs.append(TensorSpec(self.pair["name"], (int(self.pair["buckets"]) + 1, self.width), kind="table"))
         if self.projects:
@@ -95,6 +102,8 @@ class ResidualStream(Stream):
         return specs
 
     def bind(self, tensors):
+        if self.start_norm is not None:
+            self.start_norm.bind(tensors)
         if self.pair:
             self.pair_table = tensors[self.pair["name"]]
         if self.projects:
@@ -122,9 +131,12 @@ class ResidualStream(Stream):
         self._rounded = None
         if self.rounded_start and ctx.dtype != torch.float32:
             self._rounded = torch.empty((T, self.width), dtype=ctx.dtype, device=ctx.device)
+        n = self.start_norm
+        norm = {} if n is None else dict(norm_weight=n.weight32(), norm_bias=n.bias32() if hasattr(n, "bias32") else None, eps=n.eps, kind=n.kind)
         ops.embedding_pair(ctx.tokens, table, x, scale=self.scale, pair_table=self.pair_table, buckets=pair.get("buckets", 0),
                            mul_prev=pair.get("mul_prev", 0), mul_cur=pair.get("mul_cur", 0), prev_state=state, tok_row=ctx.tok_row,
-                           tok_pos=ctx.tok_pos, row_q_start=ctx.row_q_start, row_slot=ctx.row_slot, keep=keep, rounded=self._rounded, err=ctx.err)
+                           tok_pos=ctx.tok_pos, row_q_start=ctx.row_q_start, row_slot=ctx.row_slot, keep=keep, rounded=self._rounded, **norm,
+                           err=ctx.err)
         if self.pair:
             ops.remember_tokens(ctx.tokens, state, row_q_start=ctx.row_q_start, row_q_len=ctx.row_q_len, row_slot=ctx.row_slot)
         self._kept = keep
@@ -143,7 +155,7 @@ class ResidualStream(Stream):
             self._projected = linear.linear_f32(ctx, e, self.w_embed)
         h = torch.empty((T, self.width), dtype=ctx.dtype, device=x.device)
         p = pending or Pending()
-        ops.residual_norm(x, h, updates=p.updates, extra=p.extra, vec=p.vec, write_back=False)   # the settled stream, rounded once
+        ops.residual_norm(x, h, **p.sums(), write_back=False)   # the settled stream, rounded once
         return linear.linear_f32(ctx, h, self.w_stream), Pending((), self._projected, None)
 
     def enter_pass(self, ctx, x, pending, number: int):
@@ -153,10 +165,10 @@ class ResidualStream(Stream):
             return self._enter_projected(ctx, x, pending)
         p = pending or Pending()
         if p.extra is not None or p.vec is not None:      # two re-entries without a layer between them: settle the first
-            ops.residual_norm(x, None, updates=p.updates, extra=p.extra, vec=p.vec)
+            ops.residual_norm(x, None, **p.sums())
             p = Pending()
         extra = self._kept if (number > 0 and self._keeps()) else None
-        return x, Pending(p.updates, extra, self.pass_vectors[number])
+        return x, Pending(p.updates, extra, self.pass_vectors[number], p.scale)
 
     def finish(self, ctx, x, pending, norm, rows):
         return read(ctx, x, pending, norm, rows=rows, write_back=False)
@@ -181,12 +193,14 @@ class ParallelBlock(Block):
 
 @BLOCKS.register("residual_pre_norm")
 class ResidualPreNormBlock(Block):
-    """The pre-norm arrangement on the 32-bit stream; a layer may have no feed-forward (then it has no second norm either)."""
+    """The pre-norm arrangement on the 32-bit stream; a layer may have no feed-forward (then it has no second norm either).
+    ``update_scale`` multiplies every sublayer's output before it is added."""
     roles = ("norm1", "mixer")
     optional_roles = ("norm2", "feed_forward")
 
-    def __init__(self, parts):
+    def __init__(self, parts, update_scale: float = 1.0):
         super().__init__(parts)
+        self.update_scale = float(update_scale)
         if (self.norm2 is None) != (self.feed_forward is None):
             raise ValueError("the second norm and the feed-forward come together or not at all")
 
@@ -194,9 +208,9 @@ class ResidualPreNormBlock(Block):
         h = read(ctx, x, pending, self.norm1)
         y = self.mixer.forward(ctx, h, cache)
         if self.feed_forward is None:
-            return x, Pending((y,))
-        f = read(ctx, x, Pending((y,)), self.norm2)
-        return x, Pending((self.feed_forward.forward(ctx, f),))
+            return x, Pending((y,), scale=self.update_scale)
+        f = read(ctx, x, Pending((y,), scale=self.update_scale), self.norm2)
+        return x, Pending((self.feed_forward.forward(ctx, f),), scale=self.update_scale)
 
 
 @BLOCKS.register("sublayer_norm")
@@ -226,7 +240,7 @@ class SublayerNormBlock(Block):
         else:
             h = torch.empty(x.shape, dtype=ctx.dtype, device=x.device)
             p = pending or Pending()
-            ops.residual_norm(x, h, updates=p.updates, extra=p.extra, vec=p.vec)      # settles what is pending; h = x rounded once
+            ops.residual_norm(x, h, **p.sums())      # settles what is pending; h = x rounded once
         h = self._settle(ctx, x, self.mixer.forward(ctx, h, cache), self.norm1)
         if self.feed_forward is not None:
             h = self._settle(ctx, x, self.feed_forward.forward(ctx, h), self.norm2)

@@ -60,6 +60,10 @@ Other workloads (``--workload``), each printing one JSON line of the same shape:
                capped scores and biases by distance, gelu-gated feed-forwards, experts whose weights multiply their input)
                beside Yi, Pibalorn and Roletar, measured as the roletar workload is
 
+  vazunex      the Vazunex design (gated delta rule with a decay per key channel, state-space recurrence with one decay per
+               head, windowed latent attention with a sink and an output gate, experts chosen in groups, identity experts)
+               beside Yi, Mufalix, Pibalorn and Roletar, measured as the roletar workload is
+
 ``--impl reference`` runs the unmodified hoenza/DELTA engine (baseline/reference_arm.py) on the
 default workload and prints its line.
 """
@@ -459,13 +463,29 @@ def mevulix_config(d: int) -> dict:
                         dict(type="attention", mixer=att, mlp=experts)])
 
 
+def vazunex_config(d: int) -> dict:
+    """A Vazunex model with layers of the sizes of a real model of width d: state-space layers (inner width 2 d, d/32 heads of 64, 128
+    states, two groups of maps), gated delta rule layers (d/128 heads of 128, ranks of 128), latent attention (d/128 heads of 128 plain
+    and 64 rotated entries, a latent of 256, a window of 1,024); every layer with a mixture of 16 experts (4 chosen, d/2 wide each) and
+    4 identities in 4 groups of which 2 are kept."""
+    H = d // 128
+    ssd = dict(type="mamba2", mixer=dict(heads=d // 32, vdim=64, state=128, groups=2, conv=4, norm_groups=1))
+    delta = dict(type="channel_delta", mixer=dict(heads=H, kv_heads=H, dim=128, vdim=128, conv=4, decay_rank=128, gate_rank=128))
+    lat = dict(type="latent_attention", mixer=dict(heads=H, dim=128, rot_dim=64, vdim=128, kv_rank=256, scale=0.07, mask=dict(size=1024),
+                                                   rot=dict(base=500000.0, dims=64)))
+    mlp = dict(kind="moe", router=dict(experts=16, top=4, identity=4, groups=dict(count=4, keep=2), scale=2.0), expert=dict(ff=d // 2))
+    return dict(architecture="Vazunex", vocab=32000, width=d, norm=dict(eps=1e-5), logit_scale=0.5, residual_mult=0.5,
+                layers=[dict(L, mlp=mlp) for L in (ssd, delta, lat, delta, ssd, lat)])
+
+
 def roletar_workload(args) -> int:
     return design_workload(args, "roletar")
 
 
 def design_workload(args, design: str) -> int:
-    """Prefill (one prompt of 2,048 tokens in one step) and decode (batch 8 at context 2,048) of a design (Roletar, Pibalorn, Mufalix, Mevulix) beside the
-    Yi architecture at equal width and layer count (Mufalix also beside Pibalorn, the closest design; Mevulix beside Pibalorn and Roletar), through ``ModelRunner.step``, timed with CUDA events after warm-up with
+    """Prefill (one prompt of 2,048 tokens in one step) and decode (batch 8 at context 2,048) of a design (Roletar, Pibalorn, Mufalix, Mevulix, Vazunex) beside the
+    Yi architecture at equal width and layer count (Mufalix also beside Pibalorn, the closest design; Mevulix beside Pibalorn and Roletar;
+    Vazunex beside Mufalix, Pibalorn and Roletar), through ``ModelRunner.step``, timed with CUDA events after warm-up with
     the L2 flushed before every timed step; then every launcher's share of one such step, with the fraction of the measured
     peaks that the design's own kernels and their Yi counterparts reach."""
     import torch
@@ -546,16 +566,19 @@ def design_workload(args, design: str) -> int:
 
     launches = 0
     for d in args.width:
-        rc = {"roletar": roletar_config, "pibalorn": pibalorn_config, "mufalix": mufalix_config, "mevulix": mevulix_config}[design](d)
+        rc = {"roletar": roletar_config, "pibalorn": pibalorn_config, "mufalix": mufalix_config, "mevulix": mevulix_config, "vazunex": vazunex_config}[design](d)
         runs = 6
         yc = yi_like_config(d, runs)
         a, b = measure(rc, rc["vocab"]), measure(yc, yc["vocab_size"])
-        if design in ("mufalix", "mevulix"):     # the closest design of the engine (32-bit stream, layer norms, experts beside a shared one) as well
+        if design in ("mufalix", "mevulix", "vazunex"):     # the closest design of the engine (32-bit stream, layer norms, experts beside a shared one) as well
             pc = pibalorn_config(d)
             c = measure(pc, pc["vocab"])
-        if design == "mevulix":     # and the one whose mixers are the closest (latent attention, attention with a sink over a cache of rows)
+        if design in ("mevulix", "vazunex"):     # and the one whose mixers are the closest (latent attention, attention with a sink over a cache of rows)
             oc = roletar_config(d)
             c2 = measure(oc, oc["vocab"])
+        if design == "vazunex":     # recurrent mixers behind a 32-bit stream, gated norms, a windowed attention with a sink and a gate
+            mc = mufalix_config(d)
+            c3 = measure(mc, mc["vocab"])
         launches += a["launches_per_decode_step"]
         H = d // 128
         # what the kernels of one step have to move or compute, per launcher (prefill of T tokens unless said otherwise)
@@ -586,11 +609,12 @@ def design_workload(args, design: str) -> int:
             }
         if design == "pibalorn":
             work = pibalorn_work()
-        if design == "mufalix":
+
+        def mufalix_work():
             G, top, F, Wn = max(1, H // 4), 4, d // 2, 1024
             n_mem, n_pair, n_moe = 3, 3, 6          # runs of a matrix-memory layer, of a pair of mixers, of a mixture
             seen = Wn * T - Wn * (Wn - 1) // 2       # (query, key) pairs inside the window
-            work = {
+            return {
                 "residual_norm": ((2 * d * 4 + 2 * d * 4 + d * 2) * T * (2 * runs), 0),
                 "matrix_memory_chunked": (0, 2 * T * H * (2 * 128 * 128 + 16 * (128 + 128)) * n_mem),     # counted as the linear attention's
                 "gated_rms_norm": ((H * 128 * 4 + 2 * H * 128 * 2) * T * (n_mem + n_pair), 0),
@@ -603,6 +627,30 @@ def design_workload(args, design: str) -> int:
                 "experts_combine": ((top * d * 4 + d * 4) * T * n_moe, 0),
                 "experts_gemm_tc": (0, 2 * T * top * 2 * d * F * n_moe),
                 "attention_rows_mma": (0, 4 * 128 * H * seen * n_pair),
+            }
+        if design == "mufalix":
+            work = mufalix_work()
+        if design == "vazunex":
+            top, F, Hs, P, Ns, G, Wn = 4, d // 2, d // 32, 64, 128, 2, 1024
+            n_ssd, n_delta, n_lat, n_moe = 2, 2, 2, 6
+            ch = Hs * P + 2 * G * Ns                  # channels of a state-space layer's convolution
+            seen = Wn * T - Wn * (Wn - 1) // 2
+            real = 16 / 20                           # the share of the choices that are experts, when the choices are spread evenly
+            work = {
+                "residual_norm": ((2 * d * 4 + 3 * d * 2) * T * (2 * runs), 0),
+                "embedding_pair": ((d * 2 + d * 4) * T, 0),
+                "conv_silu": ((2 * ch * n_ssd + 2 * 3 * d * n_delta) * 2 * T, 0),
+                "state_space_chunked": (0, 2 * T * Hs * (2 * Ns * P + 16 * P) * n_ssd + 2 * T * G * 16 * Ns * n_ssd),
+                "delta_rule_chunked": (0, 2 * T * H * (3 * 128 * 128 + 16 * (2 * 128 + 128)) * n_delta),
+                "gated_rms_norm": ((Hs * P * (4 + 2 + 2) * n_ssd + H * 128 * (4 + 4 + 2) * n_delta) * T, 0),
+                "latent_prepare": ((H * 192 + 320 + 320 + H * 64) * 2 * T * n_lat, 0),
+                "sigmoid_gate": (3 * H * 128 * 2 * T * n_lat, 0),
+                "experts_gather": (2 * top * real * d * 2 * T * n_moe, 0),
+                "experts_combine": ((top * real * d * 4 + d * 2 + d * 4) * T * n_moe, 0),
+                "experts_gemm_tc": (0, 2 * T * top * real * 3 * d * F * n_moe),
+                "library batched product": (0, 2 * T * H * (128 * 256 + 256 * 128) * n_lat),
+                "gemm_nt_plain_batched": (0, 2 * T * H * (128 * 256 + 256 * 128) * n_lat),
+                "attention_rows_mma": (0, 2 * H * (320 + 256) * seen * n_lat),
             }
         if design == "mevulix":
             G, top, F, Fd, Rq = max(1, H // 4), 4, d // 2, (8 * d // 3 + 255) // 256 * 256, 3 * d // 8
@@ -630,6 +678,8 @@ def design_workload(args, design: str) -> int:
             "gemm_nt_plain_batched": (0, 2 * T * H * (128 * 256 + 256 * 128) * 4),
             "library batched product": (0, 2 * T * H * (128 * 256 + 256 * 128) * 4),
             "attention_rows_mma": (0, 4 * (2 * H * (320 + 256) * T * (T + 1) // 2) + 2 * H * 256 * (1024 * T - 1024 * 1023 // 2)),
+            "selective_scan": ((4 * C + 2 * N) * 2 * T, 0),
+            "conv_silu": (2 * C * 2 * T, 0),
         }
         yi_work = {
             "rms_norm": (4 * d * 2 * T * (2 * runs) , 0),
@@ -665,12 +715,17 @@ def design_workload(args, design: str) -> int:
                              "decode_ms": c["decode_ms"], "decode_graph_ms": c["decode_graph_ms"],
                              "launches_per_decode_step": c["launches_per_decode_step"],
                              "prefill_launchers": fractions(c["prefill_launchers"], pibalorn_work()),
-                             "decode_launchers": fractions(c["decode_launchers"], {})}} if design in ("mufalix", "mevulix") else {}),
+                             "decode_launchers": fractions(c["decode_launchers"], {})}} if design in ("mufalix", "mevulix", "vazunex") else {}),
+            **({"mufalix": {"prefill_tok_s": T / c3["prefill_ms"] * 1e3, "prefill_ms": c3["prefill_ms"], "decode_tok_s": B / c3["decode_ms"] * 1e3,
+                            "decode_ms": c3["decode_ms"], "decode_graph_ms": c3["decode_graph_ms"],
+                            "launches_per_decode_step": c3["launches_per_decode_step"],
+                            "prefill_launchers": fractions(c3["prefill_launchers"], mufalix_work()),
+                            "decode_launchers": fractions(c3["decode_launchers"], {})}} if design == "vazunex" else {}),
             **({"roletar": {"prefill_tok_s": T / c2["prefill_ms"] * 1e3, "prefill_ms": c2["prefill_ms"], "decode_tok_s": B / c2["decode_ms"] * 1e3,
                             "decode_ms": c2["decode_ms"], "decode_graph_ms": c2["decode_graph_ms"],
                             "launches_per_decode_step": c2["launches_per_decode_step"],
                             "prefill_launchers": fractions(c2["prefill_launchers"], roletar_work),
-                            "decode_launchers": fractions(c2["decode_launchers"], {})}} if design == "mevulix" else {}),
+                            "decode_launchers": fractions(c2["decode_launchers"], {})}} if design in ("mevulix", "vazunex") else {}),
             "config": {"width": d, "layer_runs": runs, "prefill_tokens": T, "decode_batch": B, "decode_context": CTX,
                        "l2": "flushed before every timed step"}}
     first = out["sizes"][str(args.width[0])]
@@ -696,9 +751,9 @@ def main() -> int:
     ap.add_argument("--enable_selective_cache", action="store_true", help="DELTA on (not the default run)")
     ap.add_argument("--full_cache_layers", nargs="+", type=int, default=[0, 1, 2, 14, 22])
     ap.add_argument("--subset_cache_size", type=int, default=64)
-    ap.add_argument("--workload", choices=["decode", "baseline", "yi9b-long", "yi34b-mixed", "grown", "long-prompt", "roletar", "pibalorn", "mufalix", "mevulix"],
+    ap.add_argument("--workload", choices=["decode", "baseline", "yi9b-long", "yi34b-mixed", "grown", "long-prompt", "roletar", "pibalorn", "mufalix", "mevulix", "vazunex"],
                     default="decode")
-    ap.add_argument("--width", type=int, nargs="+", default=[2048, 4096], help="--workload roletar / pibalorn / mufalix / mevulix: the model widths that are measured")
+    ap.add_argument("--width", type=int, nargs="+", default=[2048, 4096], help="--workload roletar / pibalorn / mufalix / mevulix / vazunex: the model widths that are measured")
     ap.add_argument("--generate", type=int, default=None, help="tokens generated per request in the other workloads (default: what the workload names)")
     args = ap.parse_args()
     if args.impl == "reference":
@@ -708,7 +763,7 @@ def main() -> int:
         return 2
     if args.warmup < 3:
         args.warmup = 3
-    if args.workload in ("roletar", "pibalorn", "mufalix", "mevulix"):
+    if args.workload in ("roletar", "pibalorn", "mufalix", "mevulix", "vazunex"):
         return design_workload(args, args.workload)
     if args.workload != "decode":
         return other_workload(args)

@@ -478,6 +478,52 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ o, const TG* _
   }
 }
 
+// The same for rows and groups that are multiples of 8 with 16-byte aligned addresses: eight entries a thread in registers, all
+// loads under way before the first sum.  WARP: a warp per group of up to 256 V entries (a head); else a block per row.
+template <typename T, typename TG, bool FIRST, bool WARP, int V>
+__global__ void __launch_bounds__(256) gated_norm_vec_kernel(const float* __restrict__ o, const TG* __restrict__ gate, int gate_stride,
+                                                             const float* __restrict__ w, T* __restrict__ out, int n, int group, float eps) {
+  __shared__ float scratch[34];
+  const int t = blockIdx.x, step = WARP ? 32 : blockDim.x, at = WARP ? threadIdx.x & 31 : threadIdx.x;
+  const float* x = o + (size_t)t * n;
+  const TG* gt = gate + (size_t)t * gate_stride;
+  for (int g0 = WARP ? (threadIdx.x >> 5) * group : 0; g0 < n; g0 += WARP ? (blockDim.x >> 5) * group : n) {
+    float v[V][8], g[V][8];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      const int c = (at + k * step) * 8;
+      if (c < group) {
+        load8<float>(x + g0 + c, v[k]);
+        load8<TG>(gt + g0 + c, g[k]);
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < V; ++k)
+      if ((at + k * step) * 8 < group) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          g[k][e] = FIRST ? act_silu(g[k][e]) : 1.f / (1.f + expf(-g[k][e]));
+          const float y = FIRST ? v[k][e] * g[k][e] : v[k][e];
+          ss = fmaf(y, y, ss);
+        }
+      }
+    ss = WARP ? warp_sum(ss) : block_sum(ss, scratch);
+    const float inv = 1.f / sqrtf(ss / (float)group + eps);
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      const int c = (at + k * step) * 8;
+      if (c < group) {
+        float wv[8], r[8];
+        load8<float>(w + g0 + c, wv);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) r[e] = v[k][e] * (inv * wv[e]) * g[k][e];
+        store8<T>(out + (size_t)t * n + g0 + c, r);
+      }
+    }
+  }
+}
+
 size_t smem_floats(int dk, int dvs) { return (size_t)dk * dvs + 2 * (size_t)C * (dk + 1) + (size_t)C * dvs + C * (C + 1) + C + 1; }
 constexpr size_t SMEM_LIMIT = 200 * 1024;
 }  // namespace
@@ -525,9 +571,18 @@ extern "C" int dk_gated_rms_norm(const float* o, const void* gate, int gate_stri
   DK_REQUIRE(T_ > 0 && n > 0 && gate_stride >= n, "gated_rms_norm: bad sizes T=%d n=%d stride=%d", T_, n, gate_stride);
   DK_REQUIRE(group > 0 && n % group == 0, "gated_rms_norm: groups of %d entries do not divide a row of %d", group, n);
   const int threads = n >= 2048 ? 256 : 128;
+  const int gate_align = gate_dtype == DK_F32 ? 4 : 8;
+  const bool vec = group % 8 == 0 && gate_stride % gate_align == 0 && ((uintptr_t)o % 16) == 0 && ((uintptr_t)gate % 16) == 0 &&
+                   ((uintptr_t)w % 16) == 0 && ((uintptr_t)out % 16) == 0;
+  const bool one = group <= 256, two = group <= 512, row1 = group == n && n <= 2048, row2 = group == n && n <= 4096, row4 = group == n && n <= 8192;
 #define LAUNCH(T, TG, FIRST)                                                                                                      \
   do {                                                                                                                            \
-    if (group != n) gated_group_norm_kernel<T, TG, FIRST><<<T_, threads, 0, stream>>>(o, (const TG*)gate, gate_stride, w, (T*)out, n, group, eps); \
+    if (vec && one) gated_norm_vec_kernel<T, TG, FIRST, true, 1><<<T_, threads, 0, stream>>>(o, (const TG*)gate, gate_stride, w, (T*)out, n, group, eps); \
+    else if (vec && two) gated_norm_vec_kernel<T, TG, FIRST, true, 2><<<T_, threads, 0, stream>>>(o, (const TG*)gate, gate_stride, w, (T*)out, n, group, eps); \
+    else if (vec && row1) gated_norm_vec_kernel<T, TG, FIRST, false, 1><<<T_, 256, 0, stream>>>(o, (const TG*)gate, gate_stride, w, (T*)out, n, group, eps); \
+    else if (vec && row2) gated_norm_vec_kernel<T, TG, FIRST, false, 2><<<T_, 256, 0, stream>>>(o, (const TG*)gate, gate_stride, w, (T*)out, n, group, eps); \
+    else if (vec && row4) gated_norm_vec_kernel<T, TG, FIRST, false, 4><<<T_, 256, 0, stream>>>(o, (const TG*)gate, gate_stride, w, (T*)out, n, group, eps); \
+    else if (group != n) gated_group_norm_kernel<T, TG, FIRST><<<T_, threads, 0, stream>>>(o, (const TG*)gate, gate_stride, w, (T*)out, n, group, eps); \
     else gated_rms_norm_kernel<T, TG, FIRST><<<T_, threads, 0, stream>>>(o, (const TG*)gate, gate_stride, w, (T*)out, n, eps);     \
   } while (0)
 #define BOTH(T, TG)                      \

@@ -145,6 +145,7 @@ constexpr int CP = C + 4;                // padded row of a chunk-by-chunk matri
 constexpr int PREP_THREADS = 288;        // 36 tiles of 4 x 4 token pairs on and below the diagonal, eight lanes each
 constexpr int WALK_THREADS = 256;
 constexpr int WALK_COLS = 16;            // value columns of a block
+constexpr int SHARES = WALK_THREADS / 32;      // the warps share the channels of the first product
 constexpr int WALK_LD = WALK_COLS + 4;
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr float LEAST_LOG2 = -1000.f;    // 2^-1000 is zero in 32 bit: a token's log decay is no smaller, so that sums stay finite
@@ -171,15 +172,15 @@ struct ChunkLayout {
 
 size_t prep_smem(int dk) { return (size_t)(4 * C * prep_ld(dk) + 2 * C * CP + C) * sizeof(float); }
 size_t walk_stage(int dk) { return (size_t)(2 * C * (pad_k(dk) + 4) + C * pad_k(dk) + C * WALK_LD + C * CP + pad_k(dk)) * sizeof(float); }
-size_t walk_smem(int dk, int stages) { return stages * walk_stage(dk) + (size_t)(pad_k(dk) * WALK_LD + 4 * 2 * C * WALK_LD + C * WALK_LD) * sizeof(float); }
+size_t walk_smem(int dk, int stages) { return stages * walk_stage(dk) + (size_t)(pad_k(dk) * WALK_LD + SHARES * 2 * C * WALK_LD + C * WALK_LD) * sizeof(float); }
 
 // grid (most chunks of a row, rows * H).
 template <typename T>
-__global__ void __launch_bounds__(PREP_THREADS)
+__global__ void __launch_bounds__(PREP_THREADS, 2)
 delta_chunk_kernel(const T* __restrict__ qkv, int stride, int k_off, int v_off, const T* __restrict__ b, int b_stride,
                    const float* __restrict__ a, int a_stride, const float* __restrict__ A_log, const float* __restrict__ dt_bias,
                    float* __restrict__ work, const int* __restrict__ row_q_start, const int* __restrict__ row_q_len,
-                   const int* __restrict__ chunk_base, int H, int G, int dk, int dv, float q_scale, float guard) {
+                   const int* __restrict__ chunk_base, int H, int G, int dk, int dv, float q_scale, float guard, int vec) {
   extern __shared__ __align__(16) float sm[];
   const int row = blockIdx.y / H, h = blockIdx.y % H, c0 = blockIdx.x * C, n_new = row_q_len[row];
   if (c0 >= n_new) return;
@@ -195,35 +196,51 @@ delta_chunk_kernel(const T* __restrict__ qkv, int stride, int k_off, int v_off, 
   float* Ll = Lh + C * ld;           // [C][ld]: low part
   const ChunkLayout at(dk, dv);
   float* ws = work + ((size_t)(chunk_base[row] + blockIdx.x) * H + h) * at.size;
-  for (int task = warp; task < 2 * C; task += PREP_THREADS / 32) {
-    const int t = task >> 1, which = task & 1;
-    float* dst = (which ? K : Q) + t * ld;
-    if (t < n) {
-      const T* src = qkv + (size_t)(t0 + t) * stride + (which ? k_off : 0) + (size_t)kv * dk;
-      float ss = 0.f;
-      for (int i = lane; i < dk; i += 32) {
-        const float x = to_f32<T>(src[i]);
-        dst[i] = x;
-        ss = fmaf(x, x, ss);
-      }
-      const float f = (which ? 1.f : q_scale) / sqrtf(warp_sum(ss) + guard);
-      for (int i = lane; i < dk; i += 32) dst[i] *= f;
-    } else {
-      for (int i = lane; i < dk; i += 32) dst[i] = 0.f;
-    }
-  }
   const float rate = expf(A_log[h]) * LOG2E;
-  for (int idx = tid; idx < C * dk; idx += PREP_THREADS) {
-    const int t = idx / dk, i = idx - t * dk;
-    float l = 0.f;
-    if (t < n) l = fmaxf(-rate * softplus_dr(a[(size_t)(t0 + t) * a_stride + (size_t)h * dk + i] + dt_bias[(size_t)h * dk + i]), LEAST_LOG2);
-    Lh[t * ld + i] = l;
+  if (vec) {      // sizes and addresses allow sixteen-byte loads (eight bfloat16 or float entries at a time)
+    const int per = dk / 8;
+    for (int idx = tid; idx < 2 * C * per; idx += PREP_THREADS) {
+      const int r = idx / per, i = (idx - r * per) * 8, t = r & (C - 1);
+      float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      if (t < n) load8<T>(qkv + (size_t)(t0 + t) * stride + (r < C ? 0 : k_off) + (size_t)kv * dk + i, x);
+#pragma unroll
+      for (int e = 0; e < 8; e += 2) *reinterpret_cast<float2*>(Q + r * ld + i + e) = make_float2(x[e], x[e + 1]);      // K's rows follow Q's
+    }
+    for (int idx = tid; idx < C * per; idx += PREP_THREADS) {
+      const int t = idx / per, i = (idx - t * per) * 8;
+      float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f}, bias[8];
+      if (t < n) {
+        load8<float>(a + (size_t)(t0 + t) * a_stride + (size_t)h * dk + i, x);
+        load8<float>(dt_bias + (size_t)h * dk + i, bias);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] = fmaxf(-rate * softplus_dr(x[e] + bias[e]), LEAST_LOG2);
+      }
+#pragma unroll
+      for (int e = 0; e < 8; e += 2) *reinterpret_cast<float2*>(Lh + t * ld + i + e) = make_float2(x[e], x[e + 1]);
+    }
+  } else {
+    for (int idx = tid; idx < 2 * C * dk; idx += PREP_THREADS) {
+      const int r = idx / dk, i = idx - r * dk, t = r & (C - 1);
+      Q[r * ld + i] = t < n ? to_f32<T>(qkv[(size_t)(t0 + t) * stride + (r < C ? 0 : k_off) + (size_t)kv * dk + i]) : 0.f;
+    }
+    for (int idx = tid; idx < C * dk; idx += PREP_THREADS) {
+      const int t = idx / dk, i = idx - t * dk;
+      float l = 0.f;
+      if (t < n) l = fmaxf(-rate * softplus_dr(a[(size_t)(t0 + t) * a_stride + (size_t)h * dk + i] + dt_bias[(size_t)h * dk + i]), LEAST_LOG2);
+      Lh[t * ld + i] = l;
+    }
   }
   if (tid < C) beta[tid] = tid < n ? 1.f / (1.f + expf(-to_f32<T>(b[(size_t)(t0 + tid) * b_stride + h]))) : 0.f;
   __syncthreads();
+  for (int r = warp; r < 2 * C; r += PREP_THREADS / 32) {      // unit vectors
+    float ss = 0.f;
+    for (int i = lane; i < dk; i += 32) ss = fmaf(Q[r * ld + i], Q[r * ld + i], ss);
+    const float f = (r < C ? q_scale : 1.f) / sqrtf(warp_sum(ss) + guard);
+    for (int i = lane; i < dk; i += 32) Q[r * ld + i] *= f;
+  }
   for (int i = tid; i < dk; i += PREP_THREADS) {
     double sum = 0.0;
-#pragma unroll 8
+#pragma unroll 4
     for (int t = 0; t < C; ++t) {
       sum += (double)Lh[t * ld + i];
       const float hi = (float)sum;
@@ -338,8 +355,8 @@ delta_walk_kernel(const float* __restrict__ work, float* __restrict__ state, flo
   const int stage_floats = 2 * C * wl + C * kp + C * WALK_LD + C * CP + kp;
   float* stages = sm;
   float* S = sm + STAGES * stage_floats;             // [kp][WALK_LD]
-  float* part = S + kp * WALK_LD;                    // [4][2 C][WALK_LD]: the four shares of the first product
-  float* O = part + 4 * 2 * C * WALK_LD;             // [C][WALK_LD]
+  float* part = S + kp * WALK_LD;                    // [SHARES][2 C][WALK_LD]: the shares of the first product
+  float* O = part + SHARES * 2 * C * WALK_LD;        // [C][WALK_LD]
   const int chunks = (n_new + C - 1) / C;
   const float* ws0 = work + ((size_t)chunk_base[row] * H + h) * at.size;
   auto fetch = [&](int c) {
@@ -370,7 +387,7 @@ delta_walk_kernel(const float* __restrict__ work, float* __restrict__ state, flo
     const int j = idx / kp, i = idx - j * kp;
     S[i * WALK_LD + j] = (i < dk && j < jn) ? st[(size_t)j * dk + i] : 0.f;
   }
-  const int share = tid >> 6, r = tid & 63, ti = r >> 2, tj = r & 3;
+  const int share = tid >> 5, ti = (tid & 31) >> 2, tj = tid & 3;
   for (int c = 0; c < chunks; ++c) {
     if (STAGES == 2 && c + 1 < chunks) {
       fetch(c + 1);
@@ -384,19 +401,16 @@ delta_walk_kernel(const float* __restrict__ work, float* __restrict__ state, flo
     float* U = Kd + C * kp;
     float* B = U + C * WALK_LD;
     float* D = B + C * CP;
-    {      // [W ; Q] S: rows ti, ti + 16, ti + 32, ti + 48, four columns; the channels are shared out over four groups of 64 threads
-      float acc[4][4] = {};
-#pragma unroll 2
-      for (int i4 = share; i4 < kp / 4; i4 += 4) {
-        float4 x[4], s[4];
+    {      // [W ; Q] S: a thread takes the rows ti + 8 q and four columns; the warps share the channels
+      float acc[8][4] = {};
+      for (int i4 = share; i4 < kp / 4; i4 += SHARES) {
+        float4 s[4];
 #pragma unroll
-        for (int q = 0; q < 4; ++q) {
-          x[q] = *reinterpret_cast<const float4*>(X + (ti + 16 * q) * wl + 4 * i4);
-          s[q] = *reinterpret_cast<const float4*>(S + (4 * i4 + q) * WALK_LD + 4 * tj);
-        }
+        for (int q = 0; q < 4; ++q) s[q] = *reinterpret_cast<const float4*>(S + (4 * i4 + q) * WALK_LD + 4 * tj);
 #pragma unroll
-        for (int q = 0; q < 4; ++q) {
-          const float xv[4] = {x[q].x, x[q].y, x[q].z, x[q].w};
+        for (int q = 0; q < 8; ++q) {
+          const float4 x = *reinterpret_cast<const float4*>(X + (ti + 8 * q) * wl + 4 * i4);
+          const float xv[4] = {x.x, x.y, x.z, x.w};
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             acc[q][0] = fmaf(xv[e], s[e].x, acc[q][0]);
@@ -407,15 +421,15 @@ delta_walk_kernel(const float* __restrict__ work, float* __restrict__ state, flo
         }
       }
 #pragma unroll
-      for (int q = 0; q < 4; ++q)
-        *reinterpret_cast<float4*>(part + ((size_t)share * 2 * C + ti + 16 * q) * WALK_LD + 4 * tj) = make_float4(acc[q][0], acc[q][1], acc[q][2], acc[q][3]);
+      for (int q = 0; q < 8; ++q)
+        *reinterpret_cast<float4*>(part + ((size_t)share * 2 * C + ti + 8 * q) * WALK_LD + 4 * tj) = make_float4(acc[q][0], acc[q][1], acc[q][2], acc[q][3]);
     }
     __syncthreads();
     {
       const int t = tid >> 2, j = (tid & 3) * 4;
       float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-      for (int q = 0; q < 4; ++q) {
+      for (int q = 0; q < SHARES; ++q) {
         const float4 w = *reinterpret_cast<const float4*>(part + ((size_t)q * 2 * C + t) * WALK_LD + j);
         v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
       }
@@ -557,13 +571,15 @@ extern "C" int dk_delta_rule_chunked(const void* qkv, int stride, int k_off, int
     granted[dev] = true;
   }
   const dim3 grid(max_chunks, rows * H);
+  const int vec = dk % 8 == 0 && stride % 8 == 0 && k_off % 8 == 0 && a_stride % 4 == 0 && ((uintptr_t)qkv % 16) == 0 && ((uintptr_t)a % 16) == 0 &&
+                  ((uintptr_t)dt_bias % 16) == 0;
   if (dtype == DK_F32)
     delta_chunk_kernel<float><<<grid, PREP_THREADS, prep_smem(dk), stream>>>((const float*)qkv, stride, k_off, v_off, (const float*)b, b_stride, a, a_stride,
-                                                                             A_log, dt_bias, work, row_q_start, row_q_len, chunk_base, H, G, dk, dv, q_scale, guard);
+                                                                             A_log, dt_bias, work, row_q_start, row_q_len, chunk_base, H, G, dk, dv, q_scale, guard, vec);
   else
     delta_chunk_kernel<__nv_bfloat16><<<grid, PREP_THREADS, prep_smem(dk), stream>>>((const __nv_bfloat16*)qkv, stride, k_off, v_off, (const __nv_bfloat16*)b,
                                                                                      b_stride, a, a_stride, A_log, dt_bias, work, row_q_start, row_q_len,
-                                                                                     chunk_base, H, G, dk, dv, q_scale, guard);
+                                                                                     chunk_base, H, G, dk, dv, q_scale, guard, vec);
   if (int e = dk_check_launch("delta_rule_chunked")) return e;
   const dim3 walk((dv + WALK_COLS - 1) / WALK_COLS, rows * H);
   if (walk_smem(dk, 2) <= SMEM_LIMIT)

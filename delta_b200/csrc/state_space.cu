@@ -192,9 +192,10 @@ template <typename T, int PS>
 __host__ __device__ constexpr size_t raw_bytes(int N) {
   return (size_t)(2 * TC * N + TC * PS) * sizeof(T) + (size_t)(GROUP_FLOATS + HEAD_FLOATS) * sizeof(float);
 }
+__host__ __device__ constexpr int walk_rows(int PS) { return PS / 4; }      // rows of a thread's tile in the walk's first product
 template <typename T, int PS>
 size_t walk_smem(int N) {
-  const int Np = pad4(N), ld = PS + 4, shares = WALK_THREADS / (TC / 4 * (PS / 4));
+  const int Np = pad4(N), ld = PS + 4, shares = WALK_THREADS / (TC / walk_rows(PS) * (PS / 4));
   return 2 * raw_bytes<T, PS>((N + 7) & ~7) +
          (size_t)(TC * (Np + 4) + TC * Np + TC * ld + TC * TCP + 2 * TC + Np * ld + shares * TC * ld) * sizeof(float);
 }
@@ -207,7 +208,7 @@ ssd_walk_kernel(const T* __restrict__ xbc, int stride, const float* __restrict__
                 const float* __restrict__ D, float* __restrict__ state, float* __restrict__ out, const int* __restrict__ row_slot,
                 const int* __restrict__ row_q_start, const int* __restrict__ row_q_len, const int* __restrict__ chunk_base, int H, int G,
                 int N, int P) {
-  constexpr int LD = PS + 4, JT = PS / 4, SHARE_THREADS = TC / 4 * JT, SHARES = WALK_THREADS / SHARE_THREADS;
+  constexpr int LD = PS + 4, JT = PS / 4, RT = walk_rows(PS), TI = TC / RT, SHARE_THREADS = TI * JT, SHARES = WALK_THREADS / SHARE_THREADS;
   constexpr int VN = 16 / (int)sizeof(T);      // entries of a 16-byte piece
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const int row = blockIdx.y / H, h = blockIdx.y % H, j0 = blockIdx.x * PS, n_new = row_q_len[row];
@@ -310,19 +311,16 @@ ssd_walk_kernel(const T* __restrict__ xbc, int stride, const float* __restrict__
     if (tid < TC) wo[tid] = exp2f(hs[TC + tid] + hs[2 * TC + tid]);
     const float keep = exp2f(last_h + last_l);
     __syncthreads();
-    {      // C S: rows ti + 8 q, four columns; the state entries are shared out over groups of threads
-      float acc[4][4] = {};
-#pragma unroll 2
+    {      // C S: a thread takes the rows ti + TI q and four columns; the state entries are shared out over groups of threads
+      float acc[RT][4] = {};
       for (int i4 = share; i4 < Np / 4; i4 += SHARES) {
-        float4 x[4], s[4];
+        float4 s[4];
 #pragma unroll
-        for (int q = 0; q < 4; ++q) {
-          x[q] = *reinterpret_cast<const float4*>(Cs + (ti + 8 * q) * cl + 4 * i4);
-          s[q] = *reinterpret_cast<const float4*>(S + (4 * i4 + q) * LD + 4 * tj);
-        }
+        for (int q = 0; q < 4; ++q) s[q] = *reinterpret_cast<const float4*>(S + (4 * i4 + q) * LD + 4 * tj);
 #pragma unroll
-        for (int q = 0; q < 4; ++q) {
-          const float xv[4] = {x[q].x, x[q].y, x[q].z, x[q].w};
+        for (int q = 0; q < RT; ++q) {
+          const float4 x = *reinterpret_cast<const float4*>(Cs + (ti + TI * q) * cl + 4 * i4);
+          const float xv[4] = {x.x, x.y, x.z, x.w};
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             acc[q][0] = fmaf(xv[e], s[e].x, acc[q][0]);
@@ -333,8 +331,8 @@ ssd_walk_kernel(const T* __restrict__ xbc, int stride, const float* __restrict__
         }
       }
 #pragma unroll
-      for (int q = 0; q < 4; ++q)
-        *reinterpret_cast<float4*>(part + ((size_t)share * TC + ti + 8 * q) * LD + 4 * tj) = make_float4(acc[q][0], acc[q][1], acc[q][2], acc[q][3]);
+      for (int q = 0; q < RT; ++q)
+        *reinterpret_cast<float4*>(part + ((size_t)share * TC + ti + TI * q) * LD + 4 * tj) = make_float4(acc[q][0], acc[q][1], acc[q][2], acc[q][3]);
     }
     __syncthreads();
     for (int idx = tid; idx < TC * JT; idx += WALK_THREADS) {      // the chunk's outputs
@@ -439,8 +437,8 @@ extern "C" int dk_state_space(const void* xbc, int stride, const void* dtraw, in
 
 extern "C" int dk_state_space_chunk() { return TC; }
 
-extern "C" int dk_state_space_chunked_supported(int N, int P) {
-  return N > 0 && P > 0 && chunk_smem(N) <= SMEM_LIMIT && walk_smem<float, 16>(N) <= SMEM_LIMIT;
+extern "C" int dk_state_space_chunked_supported(int N, int P, int dtype) {
+  return N > 0 && P > 0 && chunk_smem(N) <= SMEM_LIMIT && (dtype == DK_F32 ? walk_smem<float, 16>(N) : walk_smem<__nv_bfloat16, 16>(N)) <= SMEM_LIMIT;
 }
 
 // Floats of working memory per chunk.
@@ -454,7 +452,7 @@ extern "C" int dk_state_space_chunked(const void* xbc, int stride, const void* d
                                       int max_chunks, int H, int G, int N, int P, int dtype, cudaStream_t stream) {
   if (rows == 0 || max_chunks == 0) return 0;
   if (int e = check_sizes("state_space_chunked", rows, H, G, N, P)) return e;
-  DK_REQUIRE(max_chunks > 0 && total_chunks >= max_chunks && dk_state_space_chunked_supported(N, P),
+  DK_REQUIRE(max_chunks > 0 && total_chunks >= max_chunks && dk_state_space_chunked_supported(N, P, dtype),
              "state_space_chunked: heads of %d x %d do not fit the shared memory", N, P);
   DK_REQUIRE(stride >= H * P + 2 * G * N, "state_space_chunked: rows of %d elements do not hold x, B and C", stride);
   DK_REQUIRE(dtype == DK_F32 || dtype == DK_BF16, "state_space_chunked: unknown dtype %d", dtype);

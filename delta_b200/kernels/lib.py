@@ -122,7 +122,7 @@ _SIGNATURES = {
     "dk_state_space_max_state": [],
     "dk_state_space": [P, I, P, I, P, P, P, P, P, P, P, P, I, I, I, I, I, I, P],
     "dk_state_space_chunk": [],
-    "dk_state_space_chunked_supported": [I, I],
+    "dk_state_space_chunked_supported": [I, I, I],
     "dk_state_space_chunk_floats": [I, I],
     "dk_state_space_chunked": [P, I, P, I, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P],
     "dk_glu_clamped": [P, P, L, I, F, F, F, F, I, P],

@@ -1025,8 +1025,8 @@ def state_space_chunk() -> int:
     return int(_l.load().dk_state_space_chunk())
 
 
-def state_space_chunked_supported(N, P) -> bool:
-    return bool(_l.load().dk_state_space_chunked_supported(int(N), int(P)))
+def state_space_chunked_supported(N, P, dtype) -> bool:
+    return bool(_l.load().dk_state_space_chunked_supported(int(N), int(P), dtype_code(dtype)))
 
 
 def state_space_chunk_floats(H, G) -> int:

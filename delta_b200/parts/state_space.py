@@ -78,7 +78,7 @@ class StateSpace(Mixer):
         y = torch.empty((T, C), dtype=torch.float32, device=x.device)
         args = (xbc, at(self.channels + C), src.shape[1], self.A_log, self.dt_bias, self.D, st[STATE], y)
         sizes = dict(H=H, G=G, N=N, P=P)
-        if not ctx.replayable and ctx.max_q_len >= PARALLEL_FROM and ops.state_space_chunked_supported(N, P):
+        if not ctx.replayable and ctx.max_q_len >= PARALLEL_FROM and ops.state_space_chunked_supported(N, P, x.dtype):
             base, total, most = chunk_layout(ctx, ops.state_space_chunk())
             per = ops.state_space_chunk_floats(H, G)
             bound = (-(-ctx.max_step_tokens // ops.state_space_chunk()) + ctx.max_rows) * per

@@ -393,7 +393,7 @@ def test_delta_rule_kernels(dtype, decays, H, G, dk, dv):
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("decays", ["weak", "mixed", "strong"])
-@pytest.mark.parametrize("H,G,N,P", [(4, 2, 24, 16), (3, 1, 9, 14), (64, 2, 128, 64), (96, 4, 32, 40), (1, 1, 1, 1), (2, 2, 200, 33)])
+@pytest.mark.parametrize("H,G,N,P", [(4, 2, 24, 16), (3, 1, 9, 14), (64, 2, 128, 64), (96, 4, 32, 40), (1, 1, 1, 1), (2, 2, 200, 33), (1, 1, 420, 5)])
 def test_state_space_kernels(dtype, decays, H, G, N, P):
     """As for the delta rule: tokens in turn and chunks, narrow and wide slices of the channels, 16-byte copies and single loads."""
     from delta_b200.kernels import ops
@@ -424,7 +424,9 @@ def test_state_space_kernels(dtype, decays, H, G, N, P):
 
     on = dict(xbc=xbc.to(DEV), dt=dtraw.to(DEV), A_log=A_log.to(DEV), dt_bias=dt_bias.to(DEV), D=D.to(DEV))
     for chunked in (False, True):
-        assert ops.state_space_chunked_supported(N, P)
+        if chunked and not ops.state_space_chunked_supported(N, P, dtype):
+            assert N > 200
+            continue
         st = state.to(DEV).clone()
         out = torch.full((T, H * P), float("nan"), device=DEV)
         args = (on["xbc"], on["dt"].data_ptr(), H + 3, on["A_log"], on["dt_bias"], on["D"], st, out)

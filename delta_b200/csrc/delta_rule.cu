@@ -155,18 +155,22 @@ __host__ __device__ __forceinline__ int pad_k(int dk) { return (dk + 3) & ~3; }
 __host__ __device__ __forceinline__ int pad_v(int dv) { return (dv + WALK_COLS - 1) / WALK_COLS * WALK_COLS; }
 __host__ __device__ __forceinline__ int prep_ld(int dk) { return ((dk + 7) & ~7) + 2; }      // 2 mod 8: the four tiles of a warp read different banks
 
-// What delta_chunk leaves for delta_walk per (chunk, head), in floats.
+// What delta_chunk leaves for delta_walk per (chunk, head), in floats, with rows padded as the walk wants them in shared memory, so that
+// it copies one piece as it lies: W and Q (rows of wl), K (rows of kp), B (rows of CP), the decays of the whole chunk; then, per slice of
+// the value columns, U (rows of WALK_LD).
 struct ChunkLayout {
-  int w, q, k, u, b, d, size;
+  int wl, w, q, k, b, d, common, u, size;
   __host__ __device__ ChunkLayout(int dk, int dv) {
-    const int kp = pad_k(dk), vp = pad_v(dv);
+    const int kp = pad_k(dk);
+    wl = kp + 4;
     w = 0;
-    q = w + C * kp;
-    k = q + C * kp;
-    u = k + C * kp;
-    b = u + C * vp;
-    d = b + C * C;
-    size = d + kp;
+    q = w + C * wl;
+    k = q + C * wl;
+    b = k + C * kp;
+    d = b + C * CP;
+    common = d + kp;
+    u = common;
+    size = u + pad_v(dv) / WALK_COLS * C * WALK_LD;
   }
 };
 
@@ -295,7 +299,7 @@ delta_chunk_kernel(const T* __restrict__ qkv, int stride, int k_off, int v_off, 
     }
   }
   __syncthreads();
-  for (int idx = tid; idx < C * C; idx += PREP_THREADS) ws[at.b + idx] = B[(idx >> 5) * CP + (idx & 31)];
+  for (int idx = tid; idx < C * C; idx += PREP_THREADS) ws[at.b + (idx >> 5) * CP + (idx & 31)] = B[(idx >> 5) * CP + (idx & 31)];
   for (int idx = tid; idx < C * kp; idx += PREP_THREADS) {
     const int t = idx / kp, i = idx - t * kp;
     float q = 0.f, k = 0.f;
@@ -304,7 +308,7 @@ delta_chunk_kernel(const T* __restrict__ qkv, int stride, int k_off, int v_off, 
       q = Q[r] * exp2f(Lh[r] + Ll[r]);
       k = K[r] * exp2f((Lh[last] - Lh[r]) + (Ll[last] - Ll[r]));
     }
-    ws[at.q + idx] = q;
+    ws[at.q + t * at.wl + i] = q;
     ws[at.k + idx] = k;
   }
   for (int i = tid; i < kp; i += PREP_THREADS) ws[at.d + i] = i < dk ? exp2f(Lh[(C - 1) * ld + i] + Ll[(C - 1) * ld + i]) : 0.f;
@@ -333,8 +337,8 @@ delta_chunk_kernel(const T* __restrict__ qkv, int stride, int k_off, int v_off, 
         if (4 * t4 + 3 > s) r[4 * t4 + 3] = fmaf(-w.w, x, r[4 * t4 + 3]);
       }
     }
-    float* dst = c < vp ? ws + at.u + c : ws + at.w + i;
-    const int step = c < vp ? vp : kp;
+    float* dst = c < vp ? ws + at.u + (c / WALK_COLS) * C * WALK_LD + c % WALK_COLS : ws + at.w + i;
+    const int step = c < vp ? WALK_LD : at.wl;
 #pragma unroll
     for (int t = 0; t < C; ++t) dst[(size_t)t * step] = r[t];
   }
@@ -349,10 +353,10 @@ delta_walk_kernel(const float* __restrict__ work, float* __restrict__ state, flo
   extern __shared__ __align__(16) float sm[];
   const int row = blockIdx.y / H, h = blockIdx.y % H, j0 = blockIdx.x * WALK_COLS, n_new = row_q_len[row];
   if (n_new <= 0) return;
-  const int kp = pad_k(dk), vp = pad_v(dv), wl = kp + 4, tid = threadIdx.x;
-  const int jn = min(WALK_COLS, dv - j0);
   const ChunkLayout at(dk, dv);
-  const int stage_floats = 2 * C * wl + C * kp + C * WALK_LD + C * CP + kp;
+  const int kp = pad_k(dk), wl = at.wl, tid = threadIdx.x;
+  const int jn = min(WALK_COLS, dv - j0);
+  const int stage_floats = at.common + C * WALK_LD;
   float* stages = sm;
   float* S = sm + STAGES * stage_floats;             // [kp][WALK_LD]
   float* part = S + kp * WALK_LD;                    // [SHARES][2 C][WALK_LD]: the shares of the first product
@@ -362,23 +366,9 @@ delta_walk_kernel(const float* __restrict__ work, float* __restrict__ state, flo
   auto fetch = [&](int c) {
     const float* ws = ws0 + (size_t)c * H * at.size;
     float* X = stages + (STAGES == 2 ? (c & 1) : 0) * stage_floats;
-    const int k4 = kp / 4;
-    for (int idx = tid; idx < 2 * C * k4; idx += WALK_THREADS) {      // W, then the queries: rows of one matrix of 2 C rows
-      const int t = idx / k4, i = (idx - t * k4) * 4;
-      cp_async_16(smem_u32(X + t * wl + i), ws + (size_t)t * kp + i, true);
-    }
-    float* Kd = X + 2 * C * wl;
-    for (int idx = tid; idx < C * k4; idx += WALK_THREADS) cp_async_16(smem_u32(Kd + idx * 4), ws + at.k + (size_t)idx * 4, true);
-    float* U = Kd + C * kp;
-    for (int idx = tid; idx < C * (WALK_COLS / 4); idx += WALK_THREADS) {
-      const int t = idx / (WALK_COLS / 4), j = (idx - t * (WALK_COLS / 4)) * 4;
-      cp_async_16(smem_u32(U + t * WALK_LD + j), ws + at.u + (size_t)t * vp + j0 + j, true);
-    }
-    float* B = U + C * WALK_LD;
-    for (int idx = tid; idx < C * C / 4; idx += WALK_THREADS)
-      cp_async_16(smem_u32(B + (idx >> 3) * CP + (idx & 7) * 4), ws + at.b + (size_t)idx * 4, true);
-    float* D = B + C * CP;
-    for (int idx = tid; idx < k4; idx += WALK_THREADS) cp_async_16(smem_u32(D + idx * 4), ws + at.d + (size_t)idx * 4, true);
+    for (int idx = tid; idx < at.common / 4; idx += WALK_THREADS) cp_async_16(smem_u32(X + idx * 4), ws + idx * 4, true);
+    const float* u = ws + at.u + (size_t)blockIdx.x * C * WALK_LD;
+    for (int idx = tid; idx < C * WALK_LD / 4; idx += WALK_THREADS) cp_async_16(smem_u32(X + at.common + idx * 4), u + idx * 4, true);
     cp_async_commit();
   };
   fetch(0);
@@ -397,10 +387,8 @@ delta_walk_kernel(const float* __restrict__ work, float* __restrict__ state, flo
     }
     __syncthreads();
     float* X = stages + (STAGES == 2 ? (c & 1) : 0) * stage_floats;
-    float* Kd = X + 2 * C * wl;
-    float* U = Kd + C * kp;
-    float* B = U + C * WALK_LD;
-    float* D = B + C * CP;
+    const float *Kd = X + at.k, *B = X + at.b, *D = X + at.d;
+    float* U = X + at.common;
     {      // [W ; Q] S: a thread takes the rows ti + 8 q and four columns; the warps share the channels
       float acc[8][4] = {};
       for (int i4 = share; i4 < kp / 4; i4 += SHARES) {

@@ -110,7 +110,7 @@ ssd_rows_kernel(const T* __restrict__ xbc, int stride, const T* __restrict__ dtr
 constexpr int TC = 32;                   // tokens of a chunk: one lane of a warp per token when the decays are prepared
 constexpr int TCP = TC + 4;
 constexpr int CHUNK_THREADS = 128;
-constexpr int WALK_THREADS = 256;
+constexpr int WALK_THREADS = 256;       // eight threads for each of a chunk's tokens when they are fetched
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr float LEAST_LOG2 = -1000.f;    // 2^-1000 is zero in 32 bit: a token's log decay is no smaller, so that sums stay finite
 constexpr size_t SMEM_LIMIT = 220 * 1024;
@@ -232,11 +232,13 @@ ssd_walk_kernel(const T* __restrict__ xbc, int stride, const float* __restrict__
     T* rx = rc + 2 * TC * N;
     float* fl = reinterpret_cast<float*>(rx + TC * PS);
     if (VEC) {
-      const int per = N / VN;
-      for (int idx = tid; idx < 2 * TC * per; idx += WALK_THREADS) {
-        const int r = idx / per, i = (idx - r * per) * VN, t = r & (TC - 1);
-        const size_t off = (size_t)(q0 + c * TC + (t < n ? t : 0)) * stride + (size_t)H * P + (size_t)(r < TC ? G + g : g) * N + i;
-        cp_async_16(smem_u32(rc + r * N + i), xbc + off, t < n);
+      {      // eight threads a token
+        const int t = tid >> 3;
+        const T* src = xbc + (size_t)(q0 + c * TC + (t < n ? t : 0)) * stride + (size_t)H * P;
+        for (int i = (tid & 7) * VN; i < N; i += 8 * VN) {
+          cp_async_16(smem_u32(rc + t * N + i), src + (size_t)(G + g) * N + i, t < n);
+          cp_async_16(smem_u32(rc + (TC + t) * N + i), src + (size_t)g * N + i, t < n);
+        }
       }
       for (int idx = tid; idx < TC * (PS / VN); idx += WALK_THREADS) {
         const int t = idx / (PS / VN), j = (idx - t * (PS / VN)) * VN;
@@ -279,9 +281,9 @@ ssd_walk_kernel(const T* __restrict__ xbc, int stride, const float* __restrict__
     if (VEC) {
       const T* rc = piece(c);
       const T* rx = rc + 2 * TC * N;
-      for (int idx = tid; idx < TC * (N / 4); idx += WALK_THREADS) {
-        const int t = idx / (N / 4), i = (idx - t * (N / 4)) * 4;
-        const float w = exp2f((last_h - hs[TC + t]) + (last_l - hs[2 * TC + t])) * hs[t];
+      const int t = tid >> 3;      // eight threads a token
+      const float w = exp2f((last_h - hs[TC + t]) + (last_l - hs[2 * TC + t])) * hs[t];
+      for (int i = (tid & 7) * 4; i < N; i += 32) {
         const T* pc = rc + t * N + i;
         const T* pb = pc + TC * N;
         *reinterpret_cast<float4*>(Cs + t * cl + i) = make_float4(to_f32<T>(pc[0]), to_f32<T>(pc[1]), to_f32<T>(pc[2]), to_f32<T>(pc[3]));

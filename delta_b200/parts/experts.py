@@ -85,8 +85,9 @@ class Experts(FeedForward):
     def tensor_specs(self):
         p, d, F = self.prefix, self.width, self.intermediate
         specs = [TensorSpec(p + "router", (self.outputs, d))]
-        if self.has_correction:
-            specs.append(TensorSpec(p + "correction", (self.outputs,), kind="vector", init="uniform:-0.2:0.2"))
+        if self.has_correction:      # random weights: small beside the scores, which are about 1 / outputs each under a softmax over all
+            spread = 0.2 if self.scoring == "sigmoid" else 0.2 / self.outputs
+            specs.append(TensorSpec(p + "correction", (self.outputs,), kind="vector", init=f"uniform:{-spread}:{spread}"))
         for e in range(self.experts):
             specs += ([TensorSpec(f"{p}e{e}.gate", (F, d))] if self.gated else []) + [TensorSpec(f"{p}e{e}.up", (F, d)),
                                                                                      TensorSpec(f"{p}e{e}.down", (d, F))]

@@ -9,9 +9,9 @@ pages (backend.py:263, page_selector_v2.py:62-63).
 
 What differs, on purpose:
   * Layers are sorted into groups by what they keep per token (the layout of a
-    page, which the mixer declares, and the window).  A group has a pool and block tables of its own; all layers
-    of a group share a request's page ids.  A group with a window gives pages back
-    as soon as the window has passed them; the others when the request ends.
+    page, which the mixer declares, and the window or chunk).  A group has a pool and block tables of its own; all layers
+    of a group share a request's page ids.  A group with a window or chunk gives pages back
+    as soon as the window or chunk has passed them; the others when the request ends.
   * A request holds ceil(len / page_size) pages: no empty page in advance
     (the reference allocates one whenever the length reaches a page's end,
     scheduler.py:60-66).
@@ -181,14 +181,12 @@ class CacheManager:
 
     def advance(self, slot: int, new_len: int) -> None:
         """Records that the request now holds ``new_len`` tokens, and gives back the pages
-        that every later query's window has passed."""
+        that every later query's window or chunk has passed."""
         self.seq_len[slot] = new_len
         for g in self.groups.values():
-            w = g.spec.window
-            if not w:
+            if not g.spec.reach:
                 continue
-            # the next query sits at position >= new_len and reads keys > new_len - w
-            first_needed = max(0, new_len - w + 1) // g.page_size
+            first_needed = g.spec.first_needed(new_len) // g.page_size
             a = int(g.first_page[slot])
             if first_needed > a:
                 row = g.table[slot, a:first_needed]

@@ -5,11 +5,11 @@
 // per (token, head), causal, optionally a sliding window, optionally a sink in the softmax.  The faster
 // kernels of this family are checked against it.
 //
-//   s_j  = (q . k_j) * scale          for the visible keys  max(0, i - window + 1) <= j <= i
+//   s_j  = (q . k_j) * scale          for the visible keys  max(0, i - window + 1) <= j <= i  (and of i's own chunk)
 //   s_j <- softcap * tanh(s_j / softcap)                      (softcap > 0)
 //   s_j <- s_j + dist_bias[h][min(i - j, dist_max)]           (a table of biases by distance, one row a head)
 //   p_j  = exp(s_j) / (sum_j' exp(s_j') [+ exp(sink_h)])
-//   y    = sum_j p_j v_j
+//   y    = sum_j p_j v_j              (times sigmoid of the head's gate)
 #include "common.cuh"
 #include "row_attention_params.h"
 
@@ -33,7 +33,7 @@ __global__ void __launch_bounds__(CH) attention_rows_plain_kernel(const DkRowAtt
   const T* q = (const T*)p.q + (size_t)t * p.q_stride + (size_t)h * p.q_head_stride;
   const T* cache = (const T*)p.cache;
   for (int i = tid; i < dk; i += CH) qs[i] = to_f32<T>(q[i]);
-  const int lo = (p.window > 0 && pos - p.window + 1 > 0) ? pos - p.window + 1 : 0;
+  const int lo = row_first_key(p, pos);
   const int first_page = lo / ps;
   const int n_entries = pos / ps - first_page + 1;
 
@@ -99,7 +99,7 @@ __global__ void __launch_bounds__(CH) attention_rows_plain_kernel(const DkRowAtt
     __syncthreads();
   }
   T* out = (T*)p.out + ((size_t)t * p.H + h) * dv;
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  const float inv = l > 0.f ? row_head_gate<T>(p, t, h) / l : 0.f;
 #pragma unroll
   for (int dd = 0; dd < MAX_DV / CH; ++dd) {
     const int d = tid + dd * CH;
@@ -336,6 +336,8 @@ static int check_row_params(const DkRowAttnParams& p, const char* who) {
   DK_REQUIRE(p.k_off >= 0 && p.v_off >= 0 && p.k_off + p.dk <= p.row_width && p.v_off + p.dv <= p.row_width,
              "%s: key [%d, +%d) or value [%d, +%d) does not lie in a row of %d", who, p.k_off, p.dk, p.v_off, p.dv, p.row_width);
   DK_REQUIRE(p.dtype == DK_F32 || p.dtype == DK_BF16, "%s: unknown dtype %d", who, p.dtype);
+  DK_REQUIRE(p.window >= 0 && p.chunk >= 0, "%s: bad window %d or chunk %d", who, p.window, p.chunk);
+  DK_REQUIRE(p.gate == nullptr || p.gate_stride >= p.H, "%s: rows of %d gates do not hold %d heads", who, p.gate_stride, p.H);
   return 0;
 }
 

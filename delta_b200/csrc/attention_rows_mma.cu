@@ -7,7 +7,7 @@
 // read once for all of them; a single decoded token is a tile of G rows.  Keys stream through shared memory in
 // tiles (cp.async, two stages, 16-byte chunks swizzled for ldmatrix); a cached row holds key and value, so one
 // copy brings both, and a value that is the front of its key is not copied twice.  Per tile and warp:
-// S = Q K^T (mma.sync.m16n8k16, float accumulators), mask by position (causal, window), online softmax in
+// S = Q K^T (mma.sync.m16n8k16, float accumulators), mask by position (causal, window, chunk), online softmax in
 // float (scores may first be capped, s <- cap tanh(s / cap), and take a bias by distance and head), O += P V
 // with P split into two bfloat16 parts (so the softmax weights keep 16 bits of mantissa; their sum is taken in
 // float from the unrounded weights).  The sink joins the denominator when the result is finished.
@@ -57,7 +57,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_rows_mma_kernel(const Dk
   const int nrows = min(QT, M - m0);
   const int q_start = p.row_q_start[row], pos_start = p.row_pos_start[row];
   const int first_pos = pos_start + m0 / G, last_pos = pos_start + (m0 + nrows - 1) / G;
-  const int lo_tile = (p.window > 0 && first_pos - p.window + 1 > 0) ? first_pos - p.window + 1 : 0;
+  const int lo_tile = row_first_key(p, first_pos);
   const int kt_lo = lo_tile / KT, kt_hi = last_pos / KT;
   const int splits = gridDim.y, split = blockIdx.y;
   const int per = (kt_hi - kt_lo + 1 + splits - 1) / splits;
@@ -96,6 +96,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_rows_mma_kernel(const Dk
   float o[RM][NT][4];
   float m_run[RM][2], l_run[RM][2];
   int pos_r[RM][2];     // positions of this thread's query rows: rows warp*WR + rm*16 + gq and + 8
+  int lo_r[RM][2];      // and the first keys they see
   const float* bias_r[RM][2];   // and the rows of the bias table of their heads
   bool live_r[RM][2];           // whether the tile has these rows at all
   const float inv_cap = (SHAPED && p.softcap > 0.f) ? 1.f / p.softcap : 0.f;
@@ -107,6 +108,8 @@ __global__ void __launch_bounds__(WARPS * 32) attention_rows_mma_kernel(const Dk
     l_run[rm][0] = l_run[rm][1] = 0.f;
     pos_r[rm][0] = pos_start + (m0 + min(warp * WR + rm * 16 + gq, nrows - 1)) / G;
     pos_r[rm][1] = pos_start + (m0 + min(warp * WR + rm * 16 + gq + 8, nrows - 1)) / G;
+    lo_r[rm][0] = row_first_key(p, pos_r[rm][0]);
+    lo_r[rm][1] = row_first_key(p, pos_r[rm][1]);
     if constexpr (SHAPED) {
       live_r[rm][0] = warp * WR + rm * 16 + gq < nrows;
       live_r[rm][1] = warp * WR + rm * 16 + gq + 8 < nrows;
@@ -119,6 +122,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_rows_mma_kernel(const Dk
   const float sc_log2 = p.scale * LOG2E;
   const int warp_first_pos = pos_start + (m0 + min(warp * WR, nrows - 1)) / G;
   const int warp_last_pos = pos_start + (m0 + min(warp * WR + WR - 1, nrows - 1)) / G;
+  const int warp_lo = row_first_key(p, warp_first_pos);
   const int kc0 = p.k_off / 8, vc0 = p.v_off / 8;
 
   if (kt_a < kt_b) load_tile(kt_a, 0);
@@ -131,7 +135,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_rows_mma_kernel(const Dk
     const uint32_t kbase = smem_u32(kv_smem + (size_t)((kt - kt_a) % PSTAGES) * KT * ROWS);
     const uint32_t qbase = smem_u32(q_smem);
     const int kt0 = kt * KT;
-    const bool visible = warp * WR < nrows && kt0 <= warp_last_pos && (p.window <= 0 || kt0 + KT - 1 > warp_first_pos - p.window);
+    const bool visible = warp * WR < nrows && kt0 <= warp_last_pos && kt0 + KT - 1 >= warp_lo;
     if (visible) {
       float s[RM][KT / 8][4];
 #pragma unroll
@@ -189,8 +193,8 @@ __global__ void __launch_bounds__(WARPS * 32) attention_rows_mma_kernel(const Dk
               v0 = s[rm][j][c] * sc_log2;
               v1 = s[rm][j][2 + c] * sc_log2;
             }
-            if (key > pos_r[rm][0] || (p.window > 0 && key <= pos_r[rm][0] - p.window)) v0 = -INFINITY;
-            if (key > pos_r[rm][1] || (p.window > 0 && key <= pos_r[rm][1] - p.window)) v1 = -INFINITY;
+            if (key > pos_r[rm][0] || key < lo_r[rm][0]) v0 = -INFINITY;
+            if (key > pos_r[rm][1] || key < lo_r[rm][1]) v1 = -INFINITY;
             s[rm][j][c] = v0;
             s[rm][j][2 + c] = v1;
             tmax[0] = fmaxf(tmax[0], v0);
@@ -296,7 +300,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_rows_mma_kernel(const Dk
         f = mm == -INFINITY ? 0.f : exp2f(mm - mf);
         ll = ll * f + exp2f(s2 - mf);
       }
-      const float inv = ll > 0.f ? f / ll : 0.f;
+      const float inv = ll > 0.f ? f * row_head_gate<__nv_bfloat16>(p, t, head) / ll : 0.f;
       __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(p.out) + ((size_t)t * p.H + head) * dv;
 #pragma unroll
       for (int n = 0; n < NT; ++n)
@@ -320,7 +324,7 @@ __global__ void attention_rows_merge_kernel(const DkRowAttnParams p, const float
     const float ms = src[(size_t)s * (dv + 2) + dv];
     if (ms != -INFINITY) l += src[(size_t)s * (dv + 2) + dv + 1] * exp2f(ms - mf);
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  const float inv = l > 0.f ? row_head_gate<__nv_bfloat16>(p, t, head) / l : 0.f;
   __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(p.out) + ((size_t)t * p.H + head) * dv;
   for (int d = threadIdx.x; d < dv; d += blockDim.x) {
     float a = 0.f;
@@ -385,6 +389,8 @@ extern "C" int dk_attention_rows_mma(const DkRowAttnParams* pp, int max_m, int s
   DK_REQUIRE(dk_attention_rows_mma_supported(pp), "attention_rows_mma: sizes not taken (bfloat16; key and value sizes multiples of 16, value "
              "at most 256; offsets and strides multiples of 8): dk=%d dv=%d width=%d", p.dk, p.dv, p.row_width);
   DK_REQUIRE(max_m >= 1 && splits >= 1 && splits <= 65535, "attention_rows_mma: bad max_m %d or splits %d", max_m, splits);
+  DK_REQUIRE(p.window >= 0 && p.chunk >= 0, "attention_rows_mma: bad window %d or chunk %d", p.window, p.chunk);
+  DK_REQUIRE(p.gate == nullptr || p.gate_stride >= p.H, "attention_rows_mma: rows of %d gates do not hold %d heads", p.gate_stride, p.H);
   DK_REQUIRE(splits == 1 || part != nullptr, "attention_rows_mma: splits without scratch memory");
   DK_REQUIRE(p.row_q_start && p.row_q_len && p.row_pos_start && p.tok_row, "attention_rows_mma: the rows' arrays are missing");
   DK_REQUIRE((long long)p.rows * p.KV <= 65535, "attention_rows_mma: grid too large");

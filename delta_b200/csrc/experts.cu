@@ -2,6 +2,7 @@
 //
 //   glu_clamped     y = g' * sigmoid(alpha (g' + cubic g'^3)) * (u' + shift),  g' = min(g, limit), u' = clamp(u, -limit, limit)
 //                   from rows [g (F) | u (F)] (limit < 0: nothing is clamped);
+//   table_gate      y = gate(z) * e with e a part of a table's row of the token (the same activation with u = e);
 //   router          per token the router's logits z = W x in 32 bit, the `top` largest of the E experts' logits (the lowest
 //                   index among equals) and the softmax over the chosen logits only (router_topk: the choice alone, from
 //                   logits that are there already); or scores (sigmoid, or the softmax over all E) with a correction that
@@ -65,6 +66,20 @@ __global__ void glu_clamped_vec_kernel(const T* __restrict__ gu, T* __restrict__
   }
 }
 
+// A table row that the stream gates: out[t][i] = glu_value(z[t][i], table[tokens[t]][off + i]).  A token outside the table is reported
+// and gives zeros.  One block a token.
+template <typename T>
+__global__ void table_gate_kernel(const T* __restrict__ z, const int* __restrict__ tokens, const T* __restrict__ table, long long table_stride,
+                                  long long off, int vocab, T* __restrict__ y, int n, float alpha, float cubic, int* err) {
+  const int t = blockIdx.x;
+  const int tok = tokens[t];
+  const bool bad = tok < 0 || tok >= vocab;
+  if (bad && threadIdx.x == 0) dk_report(err, DK_DEV_BAD_TOKEN, t, tok, vocab);
+  const T* row = table + (size_t)(bad ? 0 : tok) * table_stride + off;
+  for (int i = threadIdx.x; i < n; i += blockDim.x)
+    y[(size_t)t * n + i] = from_f32<T>(bad ? 0.f : glu_value(to_f32<T>(z[(size_t)t * n + i]), to_f32<T>(row[i]), -1.f, alpha, 0.f, cubic));
+}
+
 // The `top` largest of z[0..E) (the lowest index among equals) and the softmax over them, by one warp.  z is the warp's own
 // copy (shared memory) and is used up: a chosen entry is set to -inf.
 __device__ void pick_top(float* z, int E, int top, int* __restrict__ choice, float* __restrict__ weight, int lane) {
@@ -105,14 +120,23 @@ __device__ void pick_top(float* z, int E, int top, int* __restrict__ choice, flo
   }
 }
 
-// Only the `keep` best of `count` equal groups of neighbouring experts can be chosen: a group's score is its largest pick (the
-// lowest group among equals), the picks of the other groups become -inf.  `best` [count] is the warp's own memory.
-__device__ void keep_groups(float* pick, float* best, int E, int count, int keep, int lane) {
+// Only the `keep` best of `count` equal groups of neighbouring experts can be chosen: a group's score is the largest of its entries of
+// `value`, or, with `top2`, the sum of its two largest (of its only one); the lowest group among equals.  The picks of the other
+// groups become -inf.  `best` [count] is the warp's own memory.
+__device__ void keep_groups(float* pick, const float* value, float* best, int E, int count, int keep, int top2, int lane) {
   const int per = E / count;
   for (int g = lane; g < count; g += 32) {
-    float m = -INFINITY;
-    for (int i = 0; i < per; ++i) m = fmaxf(m, pick[g * per + i]);
-    best[g] = m;
+    float m = -INFINITY, second = -INFINITY;
+    for (int i = 0; i < per; ++i) {
+      const float v = value[g * per + i];
+      if (v > m) {
+        second = m;
+        m = v;
+      } else if (v > second) {
+        second = v;
+      }
+    }
+    best[g] = top2 && per > 1 ? m + second : m;
   }
   __syncwarp();
   for (int j = 0; j < keep; ++j) {
@@ -206,7 +230,7 @@ template <typename T, bool VEC>
 __global__ void __launch_bounds__(ROUTER_WARPS * 32)
 router_kernel(const T* __restrict__ x, const T* __restrict__ w, float* __restrict__ logits, int* __restrict__ choice,
               float* __restrict__ weight, int T_, int d, int n_rows, int E, int top, int tpb, const float* __restrict__ correction,
-              float route_scale, int scored, int groups, int keep) {
+              float route_scale, int scored, int groups, int keep, int group_top2) {
   extern __shared__ float zs[];      // [tpb][n_rows] (scored: and [tpb][E] behind them; with groups: and [tpb][groups])
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int local = warp % tpb, share = warp / tpb, sharers = ROUTER_WARPS / tpb;
@@ -269,7 +293,9 @@ router_kernel(const T* __restrict__ x, const T* __restrict__ w, float* __restric
       if (correction != nullptr) z[e] = sc + correction[e];
     }
     __syncwarp();
-    if (groups > 0) keep_groups(z, zs + (size_t)tpb * (n_rows + E) + (size_t)local * groups, E, groups, keep, lane);
+    if (groups > 0)      // (a sum of two needs the scores themselves; a maximum is the same by the logits)
+      keep_groups(z, group_top2 && correction == nullptr ? score : z, zs + (size_t)tpb * (n_rows + E) + (size_t)local * groups, E, groups, keep,
+                  group_top2, lane);
     pick_top_scored(z, score, E, top, route_scale, scored & 1, choice + (size_t)t * top, weight + (size_t)t * top, lane);
   } else {
     pick_top(z, E, top, choice + (size_t)t * top, weight + (size_t)t * top, lane);
@@ -603,6 +629,20 @@ extern "C" int dk_glu_clamped(const void* gu, void* y, long long rows, int F, fl
   return dk_check_launch("glu_clamped");
 }
 
+extern "C" int dk_table_gate(const void* z, const int* tokens, const void* table, long long table_stride, long long off, int vocab, void* y, int T_,
+                             int n, float alpha, float cubic, int dtype, int* err, cudaStream_t stream) {
+  if (T_ == 0) return 0;
+  DK_REQUIRE(T_ > 0 && n > 0 && vocab > 0 && off >= 0 && off + n <= table_stride, "table_gate: entries [%lld, +%d) do not lie in a row of %lld", off, n,
+             table_stride);
+  const int threads = n >= 256 ? 256 : (n + 31) / 32 * 32;
+#define LAUNCH(T) table_gate_kernel<T><<<T_, threads, 0, stream>>>((const T*)z, tokens, (const T*)table, table_stride, off, vocab, (T*)y, n, alpha, cubic, err)
+  if (dtype == DK_F32) LAUNCH(float);
+  else if (dtype == DK_BF16) LAUNCH(__nv_bfloat16);
+  else DK_REQUIRE(false, "table_gate: unknown dtype %d", dtype);
+#undef LAUNCH
+  return dk_check_launch("table_gate");
+}
+
 extern "C" int dk_router_topk(const float* logits, int ld, int* choice, float* weight, int T_, int E, int top, cudaStream_t stream) {
   if (T_ == 0) return 0;
   DK_REQUIRE(T_ > 0 && E > 0 && top > 0 && top <= E && ld >= E, "router_topk: bad sizes T=%d E=%d top=%d ld=%d", T_, E, top, ld);
@@ -616,9 +656,11 @@ extern "C" int dk_router_topk(const float* logits, int ld, int* choice, float* w
 // scored == 0: the softmax over the chosen logits.  scored == 1: sigmoid scores, `correction` [E] (or null) added for the choice
 // only, weights = chosen scores / their sum * route_scale.  scored == 2: the same with weights = chosen scores * route_scale.
 // scored == 3, 4: as 1, 2 with the softmax over all E logits as scores.  groups > 0 (scored only): the experts form that many
-// equal groups of neighbours, of which the `keep` with the largest score + correction can be chosen from.
+// equal groups of neighbours, of which the `keep` with the largest score + correction can be chosen from (group_top2: those with the
+// largest sum of their two largest).
 extern "C" int dk_router(const void* x, const void* w, float* logits, int* choice, float* weight, int T_, int d, int n_rows, int E, int top,
-                         const float* correction, float route_scale, int scored, int groups, int keep, int dtype, cudaStream_t stream) {
+                         const float* correction, float route_scale, int scored, int groups, int keep, int group_top2,
+                         int dtype, cudaStream_t stream) {
   if (T_ == 0) return 0;
   DK_REQUIRE(T_ > 0 && d > 0 && E > 0 && top > 0 && top <= E && n_rows >= E, "router: bad sizes T=%d d=%d E=%d top=%d rows=%d", T_, d, E, top, n_rows);
   DK_REQUIRE(top <= MAX_TOP, "router: %d choices a token are above the %d this kernel takes", top, MAX_TOP);
@@ -633,7 +675,7 @@ extern "C" int dk_router(const void* x, const void* w, float* logits, int* choic
   DK_REQUIRE(smem <= 48 * 1024, "router: %d logits a token do not fit the shared memory", n_rows);
   const int blocks = (T_ + tpb - 1) / tpb;
   const bool vec = d % 8 == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)w % 16) == 0;
-#define LAUNCH(T, V) router_kernel<T, V><<<blocks, ROUTER_WARPS * 32, smem, stream>>>((const T*)x, (const T*)w, logits, choice, weight, T_, d, n_rows, E, top, tpb, correction, route_scale, scored, groups, keep)
+#define LAUNCH(T, V) router_kernel<T, V><<<blocks, ROUTER_WARPS * 32, smem, stream>>>((const T*)x, (const T*)w, logits, choice, weight, T_, d, n_rows, E, top, tpb, correction, route_scale, scored, groups, keep, group_top2)
   if (dtype == DK_F32) {
     if (vec) LAUNCH(float, true);
     else LAUNCH(float, false);

@@ -8,6 +8,7 @@
 //                        x <- x + m (y1 + y2)    what the last layer's sublayers gave (either may be absent), times a constant
 //                        x <- x + e              a second 32-bit stream (the embedding output, at a re-entry)
 //                        x <- x + vec            one vector for all tokens
+//                        x <- x + y3 / sqrt(mean(y3^2) + eps3) * w3      an update that is RMS-normed before it is added
 //                    then out = norm(x) * w with the layer norm without bias, (x - mean) / sqrt(var + eps), var the
 //                    mean of the squared deviations, or the RMS norm x / sqrt(mean(x^2) + eps); w == nullptr: out = x.
 //                    A bias b (or null) is added behind the weight.
@@ -83,14 +84,23 @@ __global__ void remember_tokens_kernel(const int* __restrict__ tokens, const int
 // One block per output row r (token tk = rows ? rows[r] : r); the settled row is kept in shared memory between the passes.
 template <typename T, typename TO>
 __global__ void residual_norm_kernel(float* __restrict__ X, const T* __restrict__ y1, const T* __restrict__ y2, float mult, const float* __restrict__ e,
-                                     const float* __restrict__ vec, const float* __restrict__ w, const float* __restrict__ b,
+                                     const float* __restrict__ vec, const T* __restrict__ y3, const float* __restrict__ w3, float eps3,
+                                     const float* __restrict__ w, const float* __restrict__ b,
                                      TO* __restrict__ out, const int* __restrict__ rows, int d, float eps, int kind, int write_back) {
   extern __shared__ __align__(16) float xs[];   // d floats + 33
   float* scratch = xs + d;
   const int r = blockIdx.x;
   const int tk = rows ? rows[r] : r;
   float* x = X + (size_t)tk * d;
-  float sum = 0.f;
+  float sum = 0.f, inv3 = 0.f;
+  if (y3 != nullptr) {
+    float s3 = 0.f;
+    for (int i = threadIdx.x; i < d; i += blockDim.x) {
+      const float u = to_f32<T>(y3[(size_t)tk * d + i]);
+      s3 += u * u;
+    }
+    inv3 = 1.f / sqrtf(block_sum(s3, scratch) / (float)d + eps3);
+  }
   for (int i = threadIdx.x; i < d; i += blockDim.x) {
     float v = x[i];
     if (y1 != nullptr) {
@@ -100,6 +110,7 @@ __global__ void residual_norm_kernel(float* __restrict__ X, const T* __restrict_
     }
     if (e != nullptr) v += e[(size_t)tk * d + i];
     if (vec != nullptr) v += vec[i];
+    if (y3 != nullptr) v += to_f32<T>(y3[(size_t)tk * d + i]) * inv3 * w3[i];
     if (write_back) x[i] = v;
     xs[i] = v;
     sum += v;
@@ -121,6 +132,110 @@ __global__ void residual_norm_kernel(float* __restrict__ X, const T* __restrict_
   ss = block_sum(ss, scratch);
   const float inv = 1.f / sqrtf(ss / (float)d + eps);
   for (int i = threadIdx.x; i < d; i += blockDim.x) o[i] = from_f32<TO>((xs[i] - mean) * inv * w[i] + (b != nullptr ? b[i] : 0.f));
+}
+
+// The same for a width that is a multiple of 8 with 16-byte aligned rows: a thread keeps V groups of eight entries in registers, so
+// every load of the block is under way before the first sum is needed.
+template <typename T, typename TO, int V>
+__global__ void residual_norm_vec_kernel(float* __restrict__ X, const T* __restrict__ y1, const T* __restrict__ y2, float mult,
+                                         const float* __restrict__ e, const float* __restrict__ vec, const T* __restrict__ y3,
+                                         const float* __restrict__ w3, float eps3, const float* __restrict__ w, const float* __restrict__ b,
+                                         TO* __restrict__ out, const int* __restrict__ rows, int d, float eps, int kind, int write_back) {
+  __shared__ float scratch[34];
+  const int r = blockIdx.x;
+  const int tk = rows ? rows[r] : r;
+  const size_t at = (size_t)tk * d;
+  const int groups = d / 8;
+  float xv[V][8], uv[V][8];
+  float s3 = 0.f;
+#pragma unroll
+  for (int v = 0; v < V; ++v) {
+    const int c = (threadIdx.x + v * blockDim.x) * 8;
+    if (c < groups * 8) {
+      load8<float>(X + at + c, xv[v]);
+      if (y3 != nullptr) {
+        load8<T>(y3 + at + c, uv[v]);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) s3 += uv[v][i] * uv[v][i];
+      }
+      if (y1 != nullptr) {
+        float a[8];
+        load8<T>(y1 + at + c, a);
+        if (y2 != nullptr) {
+          float a2[8];
+          load8<T>(y2 + at + c, a2);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) a[i] += a2[i];
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) xv[v][i] = fmaf(mult, a[i], xv[v][i]);
+      }
+      if (e != nullptr) {
+        float a[8];
+        load8<float>(e + at + c, a);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) xv[v][i] += a[i];
+      }
+      if (vec != nullptr) {
+        float a[8];
+        load8<float>(vec + c, a);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) xv[v][i] += a[i];
+      }
+    }
+  }
+  if (y3 != nullptr) {
+    const float inv3 = 1.f / sqrtf(block_sum(s3, scratch) / (float)d + eps3);
+#pragma unroll
+    for (int v = 0; v < V; ++v) {
+      const int c = (threadIdx.x + v * blockDim.x) * 8;
+      if (c < groups * 8) {
+        float a[8];
+        load8<float>(w3 + c, a);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) xv[v][i] += uv[v][i] * inv3 * a[i];
+      }
+    }
+  }
+  float sum = 0.f;
+#pragma unroll
+  for (int v = 0; v < V; ++v) {
+    const int c = (threadIdx.x + v * blockDim.x) * 8;
+    if (c < groups * 8) {
+      if (write_back) store8<float>(X + at + c, xv[v]);
+      if (out != nullptr && w == nullptr) store8<TO>(out + (size_t)r * d + c, xv[v]);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) sum += xv[v][i];
+    }
+  }
+  if (out == nullptr || w == nullptr) return;
+  float mean = 0.f;
+  if (kind == 1) mean = block_sum(sum, scratch) / (float)d;
+  float ss = 0.f;
+#pragma unroll
+  for (int v = 0; v < V; ++v) {
+    const int c = (threadIdx.x + v * blockDim.x) * 8;
+    if (c < groups * 8) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        xv[v][i] -= mean;
+        ss += xv[v][i] * xv[v][i];
+      }
+    }
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)d + eps);
+#pragma unroll
+  for (int v = 0; v < V; ++v) {
+    const int c = (threadIdx.x + v * blockDim.x) * 8;
+    if (c < groups * 8) {
+      float a[8], bv[8];
+      load8<float>(w + c, a);
+      if (b != nullptr) load8<float>(b + c, bv);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) xv[v][i] = xv[v][i] * inv * a[i] + (b != nullptr ? bv[i] : 0.f);
+      store8<TO>(out + (size_t)r * d + c, xv[v]);
+    }
+  }
 }
 
 // The step behind a sublayer whose OUTPUT is normed (the sublayer itself read the stream as it was):
@@ -235,25 +350,36 @@ extern "C" int dk_remember_tokens(const int* tokens, const int* row_q_start, con
   return dk_check_launch("remember_tokens");
 }
 
-extern "C" int dk_residual_norm(float* X, const void* y1, const void* y2, float mult, const float* e, const float* vec, const float* w, const float* b,
-                                void* out, const int* rows, int n_rows, int d, float eps, int kind, int write_back, int y_dtype, int out_dtype,
+extern "C" int dk_residual_norm(float* X, const void* y1, const void* y2, float mult, const float* e, const float* vec, const void* y3,
+                                const float* w3, float eps3, const float* w, const float* b, void* out, const int* rows, int n_rows, int d, float eps, int kind, int write_back, int y_dtype, int out_dtype,
                                 cudaStream_t stream) {
   if (n_rows == 0) return 0;
   DK_REQUIRE(n_rows > 0 && d > 0, "residual_norm: bad sizes rows=%d d=%d", n_rows, d);
   DK_REQUIRE(d <= 12000, "residual_norm: width %d is above the 12000 this kernel keeps in shared memory", d);
   DK_REQUIRE(kind == 0 || kind == 1, "residual_norm: unknown norm kind %d", kind);
   DK_REQUIRE(y2 == nullptr || y1 != nullptr, "residual_norm: a second update is given without a first");
+  DK_REQUIRE(y3 == nullptr || w3 != nullptr, "residual_norm: a normed update is given without its weight");
   const int threads = d >= 4096 ? 512 : (d >= 1024 ? 256 : 128);
   const size_t smem = (size_t)(d + 36) * sizeof(float);
-#define LAUNCH(T, TO)                                                                                                          \
-  residual_norm_kernel<T, TO><<<n_rows, threads, smem, stream>>>(X, (const T*)y1, (const T*)y2, mult, e, vec, w, b, (TO*)out, rows, d, eps, \
-                                                                 kind, write_back)
+  auto aligned = [](const void* q) { return q == nullptr || ((uintptr_t)q % 16) == 0; };
+  const int groups = d / 8;
+  const bool vecs = d % 8 == 0 && groups <= 2048 && aligned(X) && aligned(y1) && aligned(y2) && aligned(e) && aligned(vec) && aligned(y3) &&
+                    aligned(w3) && aligned(w) && aligned(b) && aligned(out);
+  const int vthreads = groups <= 1024 ? (groups + 31) / 32 * 32 : 1024;      // one group of eight a thread up to a width of 8,192, then two
+#define ARGS(T, TO) X, (const T*)y1, (const T*)y2, mult, e, vec, (const T*)y3, w3, eps3, w, b, (TO*)out, rows, d, eps, kind, write_back
+#define LAUNCH(T, TO)                                                                                           \
+  do {                                                                                                          \
+    if (vecs && groups <= 1024) residual_norm_vec_kernel<T, TO, 1><<<n_rows, vthreads, 0, stream>>>(ARGS(T, TO)); \
+    else if (vecs) residual_norm_vec_kernel<T, TO, 2><<<n_rows, vthreads, 0, stream>>>(ARGS(T, TO));             \
+    else residual_norm_kernel<T, TO><<<n_rows, threads, smem, stream>>>(ARGS(T, TO));                            \
+  } while (0)
   if (y_dtype == DK_F32 && out_dtype == DK_F32) LAUNCH(float, float);
   else if (y_dtype == DK_BF16 && out_dtype == DK_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);
   else if (y_dtype == DK_BF16 && out_dtype == DK_F32) LAUNCH(__nv_bfloat16, float);
   else if (y_dtype == DK_F32 && out_dtype == DK_BF16) LAUNCH(float, __nv_bfloat16);
   else DK_REQUIRE(false, "residual_norm: unsupported dtypes y=%d out=%d", y_dtype, out_dtype);
 #undef LAUNCH
+#undef ARGS
   return dk_check_launch("residual_norm");
 }
 

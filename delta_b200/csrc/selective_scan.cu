@@ -270,6 +270,23 @@ __global__ void scan_combine_kernel(const float* __restrict__ A_log, float* __re
 }
 }  // namespace
 
+// Leaves every row's last taps-1 inputs in its slot of conv_state (kernels that make the convolution's sums themselves end with it).
+extern "C" int dk_conv_state(const void* xin, int in_stride, float* conv_state, const int* row_slot, const int* row_q_start,
+                             const int* row_q_len, int rows, int C, int taps, int dtype, cudaStream_t stream) {
+  DK_REQUIRE(rows > 0 && C > 0 && in_stride >= C && taps > 1 && taps <= MAX_TAPS, "conv_state: bad sizes rows=%d C=%d stride=%d taps=%d", rows, C,
+             in_stride, taps);
+  const int threads = C >= 256 ? 256 : 128;
+  const dim3 grid(rows, (C + threads - 1) / threads);
+  DK_REQUIRE(grid.y <= 65535, "conv_state: too many channels");
+  if (dtype == DK_F32)
+    conv_state_kernel<float><<<grid, threads, 0, stream>>>((const float*)xin, in_stride, conv_state, row_slot, row_q_start, row_q_len, C, taps, nullptr);
+  else if (dtype == DK_BF16)
+    conv_state_kernel<__nv_bfloat16><<<grid, threads, 0, stream>>>((const __nv_bfloat16*)xin, in_stride, conv_state, row_slot, row_q_start, row_q_len, C,
+                                                                   taps, nullptr);
+  else DK_REQUIRE(false, "conv_state: unknown dtype %d", dtype);
+  return dk_check_launch("conv_state");
+}
+
 extern "C" int dk_conv_silu(const void* xin, int in_stride, const float* w, const float* bias, float* conv_state, void* out,
                             const int* tok_row, const int* row_slot, const int* row_q_start, const int* row_q_len, int T_,
                             int rows, int C, int taps, const float* in_bias, int act, int single, int dtype, cudaStream_t stream) {

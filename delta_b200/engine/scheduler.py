@@ -109,9 +109,9 @@ class Scheduler:
     def _fits_alone(self, n_tokens: int) -> bool:
         for g in self.cache.groups.values():
             pages = (n_tokens + g.page_size - 1) // g.page_size
-            if g.spec.window:
-                # a windowed group keeps the window and what one step adds to it
-                pages = min(pages, (g.spec.window + self.budget + g.page_size - 1) // g.page_size + 1)
+            if g.spec.reach:
+                # a group with a window (or chunk) keeps that and what one step adds to it
+                pages = min(pages, (g.spec.reach + self.budget + g.page_size - 1) // g.page_size + 1)
             if pages > g.pool.num_pages:
                 return False
         return True
@@ -190,8 +190,8 @@ class Scheduler:
         need_len = r.total_len + 1
         for g in self.cache.groups.values():
             pages = (need_len + g.page_size - 1) // g.page_size
-            if g.spec.window:
-                pages = min(pages, (g.spec.window + min(self.budget, need_len) + g.page_size - 1) // g.page_size + 1)
+            if g.spec.reach:
+                pages = min(pages, (g.spec.reach + min(self.budget, need_len) + g.page_size - 1) // g.page_size + 1)
             if pages > g.pool.free_pages:
                 return False
         return True

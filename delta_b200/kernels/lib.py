@@ -40,10 +40,11 @@ class RowAttnParams(C.Structure):
     """Mirror of ``DkRowAttnParams`` in csrc/row_attention_params.h."""
     _fields_ = [
         ("q", P), ("out", P), ("cache", P), ("block_table", P), ("tok_row", P), ("tok_pos", P), ("row_q_start", P),
-        ("row_q_len", P), ("row_pos_start", P), ("sink", P), ("dist_bias", P), ("scratch", P), ("err", P),
+        ("row_q_len", P), ("row_pos_start", P), ("sink", P), ("dist_bias", P), ("gate", P), ("scratch", P), ("err", P),
         ("T", I), ("rows", I), ("H", I), ("KV", I), ("dk", I), ("dv", I), ("ps", I), ("max_pages", I), ("num_pages", I),
         ("q_stride", I), ("q_head_stride", I), ("row_width", I), ("k_off", I), ("v_off", I), ("window", I), ("dtype", I),
-        ("splits", I), ("row_filter", I), ("scale", F), ("softcap", F), ("dist_max", I), ("reserved", I),
+        ("splits", I), ("row_filter", I), ("scale", F), ("softcap", F), ("dist_max", I), ("chunk", I),
+        ("gate_stride", I), ("reserved", I),
     ]
 
 
@@ -91,7 +92,7 @@ _SIGNATURES = {
     "dk_wait_check": [P, C.c_longlong, P],
     "dk_embedding_pair": [P, P, P, P, P, P, P, F, P, L, L, L, P, P, P, P, P, F, I, I, I, I, I, P, P],
     "dk_remember_tokens": [P, P, P, P, P, I, P],
-    "dk_residual_norm": [P, P, P, F, P, P, P, P, P, P, I, I, F, I, I, I, I, P],
+    "dk_residual_norm": [P, P, P, F, P, P, P, P, F, P, P, P, P, I, I, F, I, I, I, I, P],
     "dk_sublayer_norm_add": [P, P, P, P, P, I, I, F, I, I, I, P],
     "dk_rows_append_unit": [P, I, P, P, P, I, P, I, P, I, I, I, I, I, I, I, I, I, I, I, I, I, F, I, P, P, P, F, I, F, I, I, P, P],
     "dk_decay_attention_slice": [I, I, I, I],
@@ -126,8 +127,10 @@ _SIGNATURES = {
     "dk_state_space_chunk_floats": [I, I],
     "dk_state_space_chunked": [P, I, P, I, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P],
     "dk_glu_clamped": [P, P, L, I, F, F, F, F, I, P],
+    "dk_table_gate": [P, P, P, L, L, I, P, I, I, F, F, I, P, P],
+    "dk_rows_conv_append": [P, I, P, I, P, P, P, P, P, P, P, I, P, I, P, I, P, I, I, I, P, P, F, P, I, F] + [I] * 11 + [P, P],
     "dk_router_topk": [P, I, P, P, I, I, I, P],
-    "dk_router": [P, P, P, P, P, I, I, I, I, I, P, F, I, I, I, I, P],
+    "dk_router": [P, P, P, P, P, I, I, I, I, I, P, F, I, I, I, I, I, P],
     "dk_experts_align": [P, I, I, P, I, P, I, I, P],
     "dk_experts_gather": [P, P, I, P, I, I, P, P],
     "dk_experts_gemm_tc_supported": [I, I, I],

@@ -526,9 +526,11 @@ RowAttnParams = _l.RowAttnParams
 
 def row_attn_params(*, q, q_stride, q_head_stride, out, cache, block_table, tok_row, tok_pos, row_q_start, row_q_len,
                     row_pos_start, H, KV, dk, dv, ps, row_width, k_off, v_off, scale, window=0, sink=None, softcap=None, dist_bias=None,
-                    err=None) -> RowAttnParams:
+                    chunk=0, gate_ptr=None, gate_stride=0, err=None) -> RowAttnParams:
     """``softcap`` c: the scaled score s becomes c tanh(s / c).  ``dist_bias`` float32 [H, D + 1]: entry min(i - j, D) of a head's row
-    is added to the scores of query i and key j (after the cap; the scale does not multiply it)."""
+    is added to the scores of query i and key j (after the cap; the scale does not multiply it).  ``chunk`` C: position i sees the keys
+    j <= i with i // C == j // C.  ``gate_ptr``: the output of head h of token t is multiplied by sigmoid of the element
+    t * ``gate_stride`` + h behind this address (elements of the type of q)."""
     i32 = torch.int32
     if tuple(cache.shape[1:]) != (KV, ps, row_width) or cache.dtype != q.dtype:
         raise KernelError(f"attention_rows: cache has shape {tuple(cache.shape)} / {cache.dtype}, expected [pages, {KV}, {ps}, {row_width}] of {q.dtype}")
@@ -550,7 +552,8 @@ def row_attn_params(*, q, q_stride, q_head_stride, out, cache, block_table, tok_
     p.max_pages, p.num_pages = block_table.shape[1], cache.shape[0]
     p.q_stride, p.q_head_stride = int(q_stride), int(q_head_stride)
     p.row_width, p.k_off, p.v_off = row_width, k_off, v_off
-    p.window = int(window or 0)
+    p.window, p.chunk = int(window or 0), int(chunk or 0)
+    p.gate, p.gate_stride = gate_ptr, int(gate_stride)
     p.dtype = dtype_code(q.dtype)
     p.scale = float(scale)
     return p
@@ -652,6 +655,43 @@ def rows_append_unit(src, tok_pos, tok_row, block_table, cache, *, H, KV, dk, dv
         int(q_temp[1]) if q_temp else 0, dtype_code(src.dtype), _ptr(err, "err", i32), _stream()), "rows_append_unit")
 
 
+def rows_conv_append(src, q_out, conv_w, conv_state, tok_pos, tok_row, block_table, cache, *, row_slot, row_q_start, row_q_len, H, KV, dk, dv,
+                     ps, row_width, k_off, v_off, table=None, rot_dims=0, interleaved=True, q_norm=None, k_norm=None, eps=0.0, first=None,
+                     mix=None, single=False, err=None):
+    """``src`` [T, >= (H+KV)*dk + KV*dv] holds the projected q, k and v.  Every column goes through a causal convolution (``conv_w``
+    float32 [taps, columns], the last tap meets the current token; None: no convolution) whose earlier inputs come from ``conv_state``
+    [slots, taps-1, columns] (float32), which is left holding every row's last inputs; query and key heads then through an RMS norm
+    (``q_norm`` / ``k_norm`` float32 [dk], ``eps``; None: not) and the rotation of ``rows_append``; q goes to ``q_out`` [T, H*dk], k and v
+    to the cache.  ``first`` [T, KV*dv]: the values that a group of layers mixes; ``mix`` "first" stores this layer's there, a
+    number l takes (1 - l) v + l first.  ``single``: every row brings one token."""
+    T = src.shape[0]
+    if cache is not None and (tuple(cache.shape[1:]) != (KV, ps, row_width) or cache.dtype != src.dtype):
+        raise KernelError(f"rows_conv_append: cache has shape {tuple(cache.shape)} / {cache.dtype}, expected [pages, {KV}, {ps}, {row_width}] of {src.dtype}")
+    if table is not None and tuple(table.shape[1:]) != (rot_dims // 2, 2):
+        raise KernelError(f"rows_conv_append: table has shape {tuple(table.shape)}, expected [positions, {rot_dims // 2}, 2]")
+    columns = (H + KV) * dk + KV * dv
+    taps = conv_w.shape[0] if conv_w is not None else 0
+    if conv_w is not None and conv_w.shape[1] != columns:
+        raise KernelError(f"rows_conv_append: the convolution has {conv_w.shape[1]} channels, expected {columns}")
+    if taps > 1 and tuple(conv_state.shape[1:]) != (taps - 1, columns):
+        raise KernelError(f"rows_conv_append: the state has shape {tuple(conv_state.shape)}, expected [slots, {taps - 1}, {columns}]")
+    if tuple(q_out.shape) != (T, H * dk):
+        raise KernelError(f"rows_conv_append: the queries have shape {tuple(q_out.shape)}, expected {(T, H * dk)}")
+    if first is not None and tuple(first.shape) != (T, KV * dv):
+        raise KernelError(f"rows_conv_append: the group's first values have shape {tuple(first.shape)}, expected {(T, KV * dv)}")
+    mode = 0 if mix is None else (1 if mix == "first" else 2)
+    i32, f32 = torch.int32, torch.float32
+    _l.check(_l.load().dk_rows_conv_append(
+        _ptr(src, "src"), src.shape[1], _ptr(conv_w, "conv_w", f32), taps, _ptr(conv_state, "conv_state", f32), _ptr(q_out, "q_out", src.dtype),
+        _ptr(tok_pos, "tok_pos", i32), _ptr(tok_row, "tok_row", i32), _ptr(row_slot, "row_slot", i32), _ptr(row_q_start, "row_q_start", i32),
+        _ptr(row_q_len, "row_q_len", i32), row_slot.shape[0], _ptr(block_table, "block_table", i32),
+        block_table.shape[1] if block_table is not None else 0, _ptr(cache, "cache"), cache.shape[0] if cache is not None else 0,
+        _ptr(table, "table", f32), table.shape[0] if table is not None else 0, int(rot_dims), int(bool(interleaved)), _ptr(q_norm, "q_norm", f32),
+        _ptr(k_norm, "k_norm", f32), float(eps), _ptr(first, "first", src.dtype), mode, float(mix) if mode == 2 else 0.0, T, H, KV, dk, dv, ps,
+        row_width, k_off, v_off, int(bool(single)), dtype_code(src.dtype), _ptr(err, "err", i32), _stream()), "rows_conv_append",
+        2 if taps > 1 and not single else 1)
+
+
 # ---- a residual stream of one 32-bit copy whose sublayers run side by side ---------------------------------------
 
 NORM_KINDS = {"rms": 0, "layer": 1}
@@ -683,10 +723,11 @@ def remember_tokens(tokens, prev_state, *, row_q_start, row_q_len, row_slot):
              "remember_tokens")
 
 
-def residual_norm(X, out, *, updates=(), update_scale=1.0, extra=None, vec=None, weight=None, bias=None, eps=0.0, kind="layer", rows=None,
+def residual_norm(X, out, *, updates=(), update_scale=1.0, extra=None, vec=None, normed=None, weight=None, bias=None, eps=0.0, kind="layer", rows=None,
                   write_back=True):
     """The step between two layers on a 32-bit stream X [T, d]:  X <- X + ``update_scale`` (y1 + y2) (``updates``: none, one or two tensors
-    of the compute type), X <- X + ``extra`` (float32 [T, d]), X <- X + ``vec`` (float32 [d]), stored when ``write_back``;
+    of the compute type), X <- X + ``extra`` (float32 [T, d]), X <- X + ``vec`` (float32 [d]),
+    X <- X + rms_norm(y) * w (``normed``: (y of the compute type, w float32 [d], eps)), stored when ``write_back``;
     then ``out`` = norm(X) * weight with the layer norm without bias or the RMS norm (``weight`` None: X itself).
     ``bias`` (float32 [d]) is added behind the weight.  ``rows``: only these tokens, in this order.  ``out`` None: only the sums
     are done."""
@@ -702,10 +743,14 @@ def residual_norm(X, out, *, updates=(), update_scale=1.0, extra=None, vec=None,
     y1 = updates[0] if len(updates) > 0 else None
     y2 = updates[1] if len(updates) > 1 else None
     f32 = torch.float32
-    ydt = dtype_code(y1.dtype) if y1 is not None else (dtype_code(out.dtype) if out is not None and out.dtype != f32 else F32)
+    y3, w3, eps3 = normed if normed is not None else (None, None, 0.0)
+    if y3 is not None and (tuple(y3.shape) != (T, d) or (y1 is not None and y1.dtype != y3.dtype)):
+        raise KernelError(f"residual_norm: the normed update has shape {tuple(y3.shape)} / {y3.dtype}, the stream {(T, d)}")
+    typed = y1 if y1 is not None else y3
+    ydt = dtype_code(typed.dtype) if typed is not None else (dtype_code(out.dtype) if out is not None and out.dtype != f32 else F32)
     _l.check(_l.load().dk_residual_norm(
         _ptr(X, "X", f32), _ptr(y1, "update"), _ptr(y2, "update", y1.dtype if y1 is not None else None), float(update_scale), _ptr(extra, "extra", f32),
-        _ptr(vec, "vec", f32), _ptr(weight, "weight", f32), _ptr(bias, "bias", f32) if weight is not None else None, _ptr(out, "out"),
+        _ptr(vec, "vec", f32), _ptr(y3, "normed"), _ptr(w3, "normed weight", f32), float(eps3), _ptr(weight, "weight", f32), _ptr(bias, "bias", f32) if weight is not None else None, _ptr(out, "out"),
         _ptr(rows, "rows", torch.int32), n, d, float(eps),
         NORM_KINDS[kind], int(bool(write_back)), ydt, dtype_code(out.dtype) if out is not None else F32, _stream()), "residual_norm")
     return out
@@ -1063,6 +1108,18 @@ def glu_clamped(gate_up, out, limit=-1.0, alpha=1.702, shift=1.0, cubic=0.0):
     return out
 
 
+def table_gate(z, tokens, table, offset, out, alpha, cubic=0.0, err=None):
+    """out[t] = z sigmoid(alpha (z + cubic z^3)) * e with e the n entries from ``offset`` on of the row tokens[t] of ``table``
+    [vocab, >= offset + n]; z and ``out`` [T, n]."""
+    T, n = z.shape
+    if tuple(out.shape) != (T, n):
+        raise KernelError(f"table_gate: the output has shape {tuple(out.shape)}, expected {(T, n)}")
+    _l.check(_l.load().dk_table_gate(_ptr(z, "z"), _ptr(tokens, "tokens", torch.int32), _ptr(table, "table", z.dtype), table.shape[1], int(offset),
+                                     table.shape[0], _ptr(out, "out", z.dtype), T, n, float(alpha), float(cubic), dtype_code(z.dtype),
+                                     _ptr(err, "err", torch.int32), _stream()), "table_gate")
+    return out
+
+
 def router_topk(logits, experts, top, choice, weight):
     """Per token the ``top`` largest of the first ``experts`` columns of float32 ``logits`` and the softmax over them."""
     T = logits.shape[0]
@@ -1071,15 +1128,17 @@ def router_topk(logits, experts, top, choice, weight):
 
 
 ROUTER_SCORINGS = {"softmax": 0, "sigmoid": 1, "softmax_all": 3}
+GROUP_SCORES = {"max": 0, "top2": 1}
 
 
-def router(x, w, experts, top, logits, choice, weight, scoring="softmax", correction=None, scale=1.0, normalize=True, groups=None):
+def router(x, w, experts, top, logits, choice, weight, scoring="softmax", correction=None, scale=1.0, normalize=True, groups=None,
+           group_score="max"):
     """logits = x w^T in 32 bit ([T, rows of w]; the first ``experts`` rows are the experts'), and per token the ``top`` largest of
     the experts' logits with the softmax over them.  ``scoring`` "sigmoid": scores s = sigmoid(logit); the ``top`` largest of
     s + ``correction`` (float32 [experts] or None) are chosen; the weights are the chosen s divided by their sum (``normalize``
     False: the chosen s themselves), times ``scale``.  ``scoring`` "softmax_all": the same with s the softmax over all ``experts`` logits.
     ``groups`` (count, keep): the experts form that many equal groups of neighbours, and only those of the ``keep`` groups with the
-    largest s + correction in them can be chosen."""
+    largest s + correction in them (``group_score`` "top2": the largest sum of their two largest) can be chosen."""
     T, d = x.shape
     if scoring not in ROUTER_SCORINGS:
         raise KernelError(f"router: unknown scoring '{scoring}'")
@@ -1087,7 +1146,7 @@ def router(x, w, experts, top, logits, choice, weight, scoring="softmax", correc
                                  _ptr(weight, "weight", torch.float32), T, d, w.shape[0], int(experts), int(top),
                                  _ptr(correction, "correction", torch.float32), float(scale),
                                  ROUTER_SCORINGS[scoring] + (0 if normalize or scoring == "softmax" else 1), int(groups[0]) if groups else 0,
-                                 int(groups[1]) if groups else 0,
+                                 int(groups[1]) if groups else 0, GROUP_SCORES[group_score],
                                  dtype_code(x.dtype), _stream()), "router")
 
 

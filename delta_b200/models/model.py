@@ -50,7 +50,11 @@ class Model:
         for p in self.parts():
             specs.extend(p.tensor_specs())
         specs.append(self.spec.lm_head)
-        return specs
+        once: Dict[str, TensorSpec] = {}      # several parts may read one tensor
+        for s in specs:
+            if once.setdefault(s.name, s).shape != s.shape:
+                raise ValueError(f"two parts name the tensor '{s.name}' with different shapes")
+        return list(once.values())
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         self.embed_table = tensors[self.spec.embedding.name]

@@ -51,15 +51,19 @@ class CacheSpec:
     manager allocates ``[layers of the group, pages, *layout]`` with the page size
     in place of ``PAGE`` and knows nothing else about the contents.  Mixers with
     equal specs share a cache group (one pool of pages, one block table per
-    request); ``window`` None means every token is kept.  ``run_tokens``: the mixer reads
+    request); ``window`` None means every token is kept.  ``chunk`` C: position i reads the positions of its own
+    chunk only, i // C == j // C (None: not).  ``run_tokens``: the mixer reads
     a request's pages fastest when the pages of this many consecutive tokens follow one another
     in the pool; the pool then hands pages out in aligned runs of that length where it can
     (0: any order is as good)."""
     layout: tuple
     window: Optional[int] = None
     run_tokens: int = 0
+    chunk: Optional[int] = None
 
     def __post_init__(self):
+        if self.window and self.chunk:
+            raise ValueError("a cache keeps a window or a chunk of tokens, not both")
         if tuple(self.layout).count(PAGE) != 1:
             raise ValueError(f"a page layout names the token axis once, as PAGE: {self.layout}")
         object.__setattr__(self, "layout", tuple(self.layout))
@@ -67,8 +71,20 @@ class CacheSpec:
     def page_shape(self, page_size: int) -> tuple:
         return tuple(page_size if a == PAGE else int(a) for a in self.layout)
 
+    @property
+    def reach(self) -> Optional[int]:
+        """The most tokens a query reads, its own included (None: all of them)."""
+        return self.window or self.chunk or None
+
+    def first_needed(self, new_len: int) -> int:
+        """The first position that queries at positions >= ``new_len`` may read."""
+        if self.window:      # the next query reads keys > new_len - window
+            return max(0, new_len - self.window + 1)
+        return new_len // self.chunk * self.chunk if self.chunk else 0
+
     def describe(self) -> str:
-        return "x".join("P" if a == PAGE else str(a) for a in self.layout) + (f"w{self.window}" if self.window else "")
+        return ("x".join("P" if a == PAGE else str(a) for a in self.layout) + (f"w{self.window}" if self.window else "")
+                + (f"c{self.chunk}" if self.chunk else ""))
 
 
 @dataclass(frozen=True)
@@ -147,6 +163,14 @@ class RunState:
 
 class FeedForward(Part):
     """``forward(ctx, x)``: rows [T, d] to rows [T, d], token by token."""
+
+    def forward(self, ctx, x):
+        raise NotImplementedError
+
+
+class TokenInput(Part):
+    """What a layer takes from the step's tokens themselves, beside the embedding.  ``forward(ctx, x)`` reads the settled stream x [T, d] in
+    the compute type and returns (y, weight, eps): y [T, d] joins the stream through an RMS norm with this float32 weight."""
 
     def forward(self, ctx, x):
         raise NotImplementedError
@@ -266,16 +290,17 @@ FEED_FORWARDS = Registry("feed-forward")
 BLOCKS = Registry("block")
 STREAMS = Registry("residual stream")
 STREAM_MIXINGS = Registry("stream mixing")
+TOKEN_INPUTS = Registry("token input")
 
 
 REGISTRIES = {"norm": NORMS, "position": POSITION_ENCODINGS, "mixer": MIXERS, "feed_forward": FEED_FORWARDS,
-              "block": BLOCKS, "stream": STREAMS, "stream_mixing": STREAM_MIXINGS}
+              "block": BLOCKS, "stream": STREAMS, "stream_mixing": STREAM_MIXINGS, "token_input": TOKEN_INPUTS}
 
 
 @dataclass(frozen=True)
 class PartSpec:
     """Registry name of a part, its parameters, and the registry it is looked up in
-    ("norm", "position", "mixer", "feed_forward", "block", "stream", "stream_mixing")."""
+    ("norm", "position", "mixer", "feed_forward", "block", "stream", "stream_mixing", "token_input")."""
     kind: str
     params: dict = field(default_factory=dict)
     category: str = ""

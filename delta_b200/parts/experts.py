@@ -12,8 +12,8 @@ by side (``csrc/gemm_tc.cu``).  The router's rows and
 the shared expert's gate row are one matrix, so one product gives both.
 
 Options: ``scoring`` "softmax_all": as "sigmoid" below with s = the softmax over all of the router's logits.  ``groups`` (count, keep): the
-router's outputs form that many equal groups of neighbours; a group's score is the largest s + correction in it, and only outputs of the
-``keep`` best groups can be chosen.  ``identity`` n: the router has n more outputs than there are experts, the last ones; a token that
+router's outputs form that many equal groups of neighbours; a group's score is the largest s + correction in it (``group_score`` "top2":
+the sum of its two largest, or its only one), and only outputs of the ``keep`` best groups can be chosen.  ``identity`` n: the router has n more outputs than there are experts, the last ones; a token that
 chooses one of them gets its own input h times the weight (no tensors, no product).  ``scoring`` "sigmoid": scores s = sigmoid(z); the ``top`` largest of s + correction (a tensor ``correction`` [E] when
 ``correction`` is set) are chosen, and the weights are the chosen s (without the correction) divided by their sum (+ 1e-20), times
 ``route_scale``; ``normalize`` False: the chosen s themselves, times ``route_scale``.  ``weight_input``: a choice's weight multiplies
@@ -45,11 +45,14 @@ class Experts(FeedForward):
     def __init__(self, prefix: str, width: int, experts: int, top: int, intermediate: int, limit=None, alpha: float = 1.702,
                  shift: float = 1.0, shared: Optional[dict] = None, scoring: str = "softmax", correction: bool = False,
                  route_scale: float = 1.0, activation: str = "clamped_glu", wide_output: bool = False, normalize: bool = True,
-                 weight_input: bool = False, identity: int = 0, groups: Optional[tuple] = None):
+                 weight_input: bool = False, identity: int = 0, groups: Optional[tuple] = None, group_score: str = "max"):
         self.prefix, self.width = prefix, int(width)
         self.experts, self.top, self.intermediate = int(experts), int(top), int(intermediate)
         self.identity, self.outputs = int(identity), int(experts) + int(identity)      # the router's outputs: experts, then identities
         self.groups = (int(groups[0]), int(groups[1])) if groups else None
+        if group_score not in ops.GROUP_SCORES:
+            raise ValueError(f"unknown score of a group '{group_score}' ({', '.join(ops.GROUP_SCORES)})")
+        self.group_score = group_score
         if not (1 <= self.top <= self.outputs):
             raise ValueError(f"{self.top} of {self.experts} experts cannot be chosen")
         if limit is not None and float(limit) < 0:
@@ -115,7 +118,7 @@ class Experts(FeedForward):
         choice = torch.empty((T, top), dtype=i32, device=dev)
         weight = torch.empty((T, top), dtype=f32, device=dev)
         ops.router(x, self.w_router, self.outputs, top, z, choice, weight, scoring=self.scoring, correction=self.correction, scale=self.route_scale,
-                   normalize=self.normalize, groups=self.groups)
+                   normalize=self.normalize, groups=self.groups, group_score=self.group_score)
         act = "gated" if self.gated else "relu_squared"
         slots = T * top
         # weight_input: a slot's weight goes into the first product (or into the gathered rows), and the sum at the end has none

@@ -87,6 +87,7 @@ class ClampedGLU(FeedForward):
         if limit is not None and float(limit) < 0:
             raise ValueError(f"a clamp at {limit} is no limit")
         self.limit, self.alpha, self.shift, self.cubic = (-1.0 if limit is None else float(limit)), float(alpha), float(shift), float(cubic)
+        self.is_silu = limit is None and dict(alpha=self.alpha, shift=self.shift, cubic=self.cubic) == SILU_GATE
         self.w_gate_up = self.w_down = None
 
     def tensor_specs(self):
@@ -99,6 +100,10 @@ class ClampedGLU(FeedForward):
         self.w_down = tensors[p + "down"]
 
     def forward(self, ctx, x):
+        if self.is_silu:      # the gate in the product's epilogue where the batch is small enough
+            act = linear.swiglu_linear(ctx, x, self.w_gate_up)
+            if act is not None:
+                return linear.linear(ctx, act, self.w_down)
         gu = linear.linear(ctx, x, self.w_gate_up)
         act = torch.empty((x.shape[0], self.intermediate), dtype=x.dtype, device=x.device)
         ops.glu_clamped(gu, act, self.limit, self.alpha, self.shift, self.cubic)

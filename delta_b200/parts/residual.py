@@ -20,7 +20,8 @@ next norm adds, so the sum costs no kernel.
 feed-forward may be absent.
 
 ``residual_pre_norm`` block: x <- x + m mixer(norm1(x)); x <- x + m feed_forward(norm2(x)) with a constant m (``update_scale``, 1
-unless given); the second sublayer may be absent.
+unless given); the second sublayer may be absent.  A layer may have a token input behind them (``parts/token_input.py``), which
+reads the stream itself: x <- x + rms_norm(token_input(x)).
 
 ``sublayer_norm`` block: the norms sit on the sublayers' outputs and the sublayers read the stream itself,
 x <- x + norm1(mixer(x)); x <- x + norm2(feed_forward(x)) (a norm may carry a scale per column behind it, "layer scale"); the second
@@ -50,15 +51,16 @@ class Pending:
     extra: Optional[torch.Tensor] = None      # float32 [T, d]
     vec: Optional[torch.Tensor] = None        # float32 [d]
     scale: float = 1.0                        # the constant that multiplies the updates
+    normed: Optional[tuple] = None            # (y [T, d], weight, eps): an update that goes through an RMS norm first (a layer's token input)
     rounded: Optional[torch.Tensor] = None    # the settled stream in the compute type, when nothing above is pending and a kernel
                                               # made it on its way (a block whose sublayers read the stream itself takes it)
 
     def sums(self) -> dict:
         """What ``ops.residual_norm`` is to add."""
-        return dict(updates=self.updates, update_scale=self.scale, extra=self.extra, vec=self.vec)
+        return dict(updates=self.updates, update_scale=self.scale, extra=self.extra, vec=self.vec, normed=self.normed)
 
     def empty(self) -> bool:
-        return not self.updates and self.extra is None and self.vec is None
+        return not self.updates and self.extra is None and self.vec is None and self.normed is None
 
 
 def read(ctx, x, pending: Optional[Pending], norm, rows=None, write_back=True):
@@ -168,7 +170,7 @@ class ResidualStream(Stream):
             ops.residual_norm(x, None, **p.sums())
             p = Pending()
         extra = self._kept if (number > 0 and self._keeps()) else None
-        return x, Pending(p.updates, extra, self.pass_vectors[number], p.scale)
+        return x, Pending(p.updates, extra, self.pass_vectors[number], p.scale, p.normed)
 
     def finish(self, ctx, x, pending, norm, rows):
         return read(ctx, x, pending, norm, rows=rows, write_back=False)
@@ -194,9 +196,9 @@ class ParallelBlock(Block):
 @BLOCKS.register("residual_pre_norm")
 class ResidualPreNormBlock(Block):
     """The pre-norm arrangement on the 32-bit stream; a layer may have no feed-forward (then it has no second norm either).
-    ``update_scale`` multiplies every sublayer's output before it is added."""
+    ``update_scale`` multiplies every sublayer's output before it is added; a token input has a norm of its own instead."""
     roles = ("norm1", "mixer")
-    optional_roles = ("norm2", "feed_forward")
+    optional_roles = ("norm2", "feed_forward", "token_input")
 
     def __init__(self, parts, update_scale: float = 1.0):
         super().__init__(parts)
@@ -207,10 +209,15 @@ class ResidualPreNormBlock(Block):
     def forward(self, ctx, x, pending, cache):
         h = read(ctx, x, pending, self.norm1)
         y = self.mixer.forward(ctx, h, cache)
-        if self.feed_forward is None:
-            return x, Pending((y,), scale=self.update_scale)
-        f = read(ctx, x, Pending((y,), scale=self.update_scale), self.norm2)
-        return x, Pending((self.feed_forward.forward(ctx, f),), scale=self.update_scale)
+        pending = Pending((y,), scale=self.update_scale)
+        if self.feed_forward is not None:
+            f = read(ctx, x, pending, self.norm2)
+            pending = Pending((self.feed_forward.forward(ctx, f),), scale=self.update_scale)
+        if self.token_input is None:
+            return x, pending
+        h = torch.empty(x.shape, dtype=ctx.dtype, device=x.device)
+        ops.residual_norm(x, h, **pending.sums())      # settles what is pending; h = x rounded once
+        return x, Pending(normed=self.token_input.forward(ctx, h))
 
 
 @BLOCKS.register("sublayer_norm")

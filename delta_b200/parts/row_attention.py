@@ -29,7 +29,17 @@ key-value head h // (H / kv_heads)), with the options
     key j (after the cap; the scale does not multiply it), with bucket(n) = n below rows/2 and
     min(rows - 1, rows/2 + floor(ln(n / (rows/2)) / ln(far / (rows/2)) * (rows - rows/2))) from there on (``distance_buckets``);
   * ``shared_kv``: the layer has no key and value projections (nor their biases and norm); it reads the cache that another layer's
-    run filled (the model's run order says which), with queries, sink and everything else of its own.
+    run filled (the model's run order says which), with queries, sink and everything else of its own;
+  * ``conv`` n: every column of q, k and v goes through a causal convolution of n taps over time directly behind the projection, before
+    norm and rotation (``<name>.conv`` [columns, n], no activation; zeros before a request's start).  The last n - 1 projected rows of a
+    request are state of the run (``conv``);
+  * ``chunk`` C: position i sees the keys j <= i of its own chunk, i // C == j // C, chunks counted from the request's start;
+  * ``value_mix`` {group, first}: the layers of a group mix the values of the group's first layer (``first`` True) into their own,
+    v <- (1 - l) v + l v_first with the learned number l = ``vmix``; the mixed v is cached.  v_first is the first layer's v of the same tokens,
+    behind its convolution;
+  * ``head_gate``: the output of head h is multiplied by one number, sigmoid((W_g h)_h) (``g`` [heads, width]), in the attention kernels.
+The options ``conv`` and ``value_mix`` share a kernel (``csrc/rows_conv.cu``) that goes from the projected rows to finished queries and cache
+rows in one pass.
 Scores and softmax weights are 32 bit in every kernel of the family.  ``run`` chooses the kernels for a batch.
 """
 from __future__ import annotations
@@ -41,12 +51,14 @@ import torch
 
 from ..kernels import ops
 from . import linear
-from .base import MIXERS, PAGE, POSITION_ENCODINGS, CacheSpec, Mixer, PartSpec, TensorSpec
+from .base import MIXERS, PAGE, POSITION_ENCODINGS, CacheSpec, Mixer, PartSpec, StateSpec, TensorSpec
 
 
 MAX_SPLITS = 32
 SINGLE_WARP_BLOCKS_PER_SM = 6      # blocks of one warp (a tile of a single token's heads) that an SM holds at a time
 PARTIALS = "row_attention.partials"
+CONV_STATE = "conv"
+FIRST_VALUES = "row_attention.first_values."
 
 
 def plain(ctx) -> bool:
@@ -82,7 +94,8 @@ def run(ctx, params) -> None:
         if not several:
             replay = getattr(ctx, "replayable", False)
             longest = ctx.cache.max_seq_len if replay else ctx.max_seq_len
-            max_keys = min(longest, params.window + 64) if params.window else longest
+            reach = params.window or params.chunk
+            max_keys = min(longest, reach + 64) if reach else longest
             rows = params.rows
             splits = decode_splits(rows, params.KV, group, max_keys, ctx.sm_count)
             if splits > 1:
@@ -108,12 +121,13 @@ def distance_buckets(rows: int, far: float) -> list:
 
 
 def make_params(ctx, *, q, q_stride, q_head_stride, out, cache, H, KV, dk, dv, row_width, k_off, v_off, scale, window=None,
-                sink=None, softcap=None, dist_bias=None):
+                sink=None, softcap=None, dist_bias=None, chunk=None, gate_ptr=None, gate_stride=0):
     return ops.row_attn_params(
         q=q, q_stride=q_stride, q_head_stride=q_head_stride, out=out, cache=cache.pages, block_table=cache.block_table,
         tok_row=ctx.tok_row, tok_pos=ctx.tok_pos, row_q_start=ctx.row_q_start, row_q_len=ctx.row_q_len,
         row_pos_start=ctx.row_pos_start, H=H, KV=KV, dk=dk, dv=dv, ps=cache.page_size, row_width=row_width, k_off=k_off,
-        v_off=v_off, scale=scale, window=window or 0, sink=sink, softcap=softcap, dist_bias=dist_bias, err=ctx.err)
+        v_off=v_off, scale=scale, window=window or 0, sink=sink, softcap=softcap, dist_bias=dist_bias, chunk=chunk or 0,
+        gate_ptr=gate_ptr, gate_stride=gate_stride, err=ctx.err)
 
 
 @MIXERS.register("sink_attention")
@@ -126,7 +140,8 @@ class SinkAttention(Mixer):
                  sink_logit: Optional[float] = None, unit_norm_eps: Optional[float] = None, value_from_key: bool = False,
                  bias: bool = False, qk_norm_eps: Optional[float] = None, gate: bool = False, wide_output: bool = False,
                  out_bias: bool = True, qk_norm_whole: bool = False, q_temp: Optional[dict] = None, softcap: Optional[float] = None,
-                 distance_bias: Optional[dict] = None, shared_kv: bool = False):
+                 distance_bias: Optional[dict] = None, shared_kv: bool = False, conv: int = 0, chunk: Optional[int] = None,
+                 value_mix: Optional[dict] = None, head_gate: bool = False):
         if heads % kv_heads:
             raise ValueError(f"{heads} heads are no multiple of {kv_heads} key-value heads")
         self.prefix, self.width = prefix, int(width)
@@ -153,6 +168,17 @@ class SinkAttention(Mixer):
         self.shared_kv = bool(shared_kv)
         if self.shared_kv and (value_from_key or gate):
             raise ValueError("a layer that reads another layer's keys and values has neither of its own to derive anything from")
+        self.taps, self.chunk, self.head_gate = int(conv), (int(chunk) if chunk else None), bool(head_gate)
+        self.value_mix = dict(group=str(value_mix["group"]), first=bool(value_mix["first"])) if value_mix else None
+        self.conv_path = self.taps > 0 or self.value_mix is not None
+        if self.conv_path and (bias or value_from_key or qk_norm_whole or q_temp or shared_kv or unit_norm_eps is not None):
+            raise ValueError("a convolution or value mixing beside biases, unit norms, norms over all heads, a query temperature, values taken "
+                             "from keys or another layer's cache is not built")
+        if self.chunk and self.window:
+            raise ValueError("a window and chunks exclude one another")
+        if self.head_gate and self.has_gate:
+            raise ValueError("a gate per head and one per entry exclude one another")
+        self.conv_w, self.mix = None, None
         self.dist_table = None
         self.fold_out_bias = False      # set by a container that adds the output bias itself (``out_bias``) in a kernel of its own
         self.in_bias = self.out_bias = self.q_norm = self.k_norm = None
@@ -163,7 +189,7 @@ class SinkAttention(Mixer):
         self.scale = float(scale) if scale is not None else 1.0 / math.sqrt(self.dk)
         self.position = position.build(POSITION_ENCODINGS) if position is not None else None
         self.rot_dims = int(rot_dims) if rot_dims else (self.dk if position is not None else 0)
-        self.names = dict(q="q", k="k", v="v", o="o", sink="sink", g="g", rel="rel")
+        self.names = dict(q="q", k="k", v="v", o="o", sink="sink", g="g", rel="rel", vmix="vmix")
         self.names.update(names or {})
         self.w_qkv = self.w_o = self.sink = None
 
@@ -181,6 +207,13 @@ class SinkAttention(Mixer):
             specs.append(TensorSpec(p + n["sink"], (self.heads,), kind="vector", init="uniform:-1:1"))
         if self.has_gate:
             specs.append(TensorSpec(p + n["g"], (self.heads * self.dv, d)))
+        if self.head_gate:
+            specs.append(TensorSpec(p + n["g"], (self.heads, d)))
+        if self.taps:
+            for k, c in (("q", self.heads * self.dk), ("k", self.kv_heads * self.dk), ("v", self.kv_heads * self.dv)):
+                specs.append(TensorSpec(p + n[k] + ".conv", (c, self.taps), kind="vector", init="uniform:-0.5:0.5"))
+        if self.value_mix and not self.value_mix["first"]:
+            specs.append(TensorSpec(p + n["vmix"], (), kind="vector", init="uniform:0:1"))
         if self.has_bias:
             specs.append(TensorSpec(p + n["q"] + ".b", (self.heads * self.dk,), kind="vector", init="uniform:-0.1:0.1"))
             if own_kv:
@@ -205,7 +238,13 @@ class SinkAttention(Mixer):
         mats = [tensors[p + n["q"]]] + ([tensors[p + n["k"]]] if own_kv else []) + ([tensors[p + n["v"]]] if has_v else [])
         if self.has_gate:      # the gate's rows ride behind q, k and v in one product
             mats.append(tensors[p + n["g"]])
-        self.w_qkv = torch.cat(mats, dim=0).contiguous()
+        if self.head_gate:
+            mats.append(tensors[p + n["g"]])
+        self.w_qkv = linear.padded_rows(torch.cat(mats, dim=0)) if self.head_gate else torch.cat(mats, dim=0).contiguous()
+        if self.taps:      # [taps, columns]: neighbouring columns side by side
+            self.conv_w = torch.cat([tensors[p + n[k] + ".conv"].float() for k in ("q", "k", "v")], dim=0).t().contiguous()
+        if self.value_mix:
+            self.mix = "first" if self.value_mix["first"] else float(tensors[p + n["vmix"]])
         if self.has_bias:
             parts = [tensors[p + n["q"] + ".b"]] + ([tensors[p + n["k"] + ".b"]] if own_kv else []) + ([tensors[p + n["v"] + ".b"]] if has_v else [])
             self.in_bias = torch.cat([t.float() for t in parts]).contiguous()
@@ -224,7 +263,10 @@ class SinkAttention(Mixer):
 
     def cache_spec(self):
         # a page of a layer: [kv head][offset in the page][key | value]
-        return CacheSpec((self.kv_heads, PAGE, self.dk + self.dv), self.window, run_tokens=128)
+        return CacheSpec((self.kv_heads, PAGE, self.dk + self.dv), self.window, run_tokens=128, chunk=self.chunk)
+
+    def run_state_specs(self):
+        return {CONV_STATE: StateSpec((self.taps - 1, (self.heads + self.kv_heads) * self.dk + self.kv_heads * self.dv))} if self.taps > 1 else {}
 
     def forward(self, ctx, x, cache):
         H, KV, dk, dv = self.heads, self.kv_heads, self.dk, self.dv
@@ -235,7 +277,17 @@ class SinkAttention(Mixer):
         append = dict(H=H, KV=0 if self.shared_kv else KV, dk=dk, dv=dv, ps=cache.page_size, row_width=dk + dv, k_off=0, v_off=dk,
                       table=table, rot_dims=self.rot_dims, interleaved=bool(getattr(self.position, "interleaved", True)), err=ctx.err)
         pages = cache.pages if cache.writes else None
-        if (self.unit_norm_eps is not None or self.value_from_key or self.has_bias or self.qk_norm_eps is not None or self.q_temp
+        q = qkv
+        if self.conv_path:
+            q = torch.empty((x.shape[0], H * dk), dtype=x.dtype, device=x.device)
+            first = None
+            if self.value_mix:      # filled by the group's first layer in this step, read by the later ones
+                first = ctx.scratch(FIRST_VALUES + self.value_mix["group"], (x.shape[0], KV * dv), x.dtype, bound=(ctx.max_step_tokens, KV * dv))
+            ops.rows_conv_append(qkv, q, self.conv_w, cache.state[CONV_STATE] if self.taps > 1 else None, ctx.tok_pos, ctx.tok_row,
+                                 cache.block_table, pages, row_slot=ctx.row_slot, row_q_start=ctx.row_q_start, row_q_len=ctx.row_q_len,
+                                 q_norm=self.q_norm, k_norm=self.k_norm, eps=self.qk_norm_eps or 0.0, first=first, mix=self.mix,
+                                 single=ctx.decode_only, **append)
+        elif (self.unit_norm_eps is not None or self.value_from_key or self.has_bias or self.qk_norm_eps is not None or self.q_temp
                 or self.shared_kv):
             ops.rows_append_unit(qkv, ctx.tok_pos, ctx.tok_row, cache.block_table, pages, unit_eps=self.unit_norm_eps,
                                  value_from_key=self.value_from_key, bias=self.in_bias, q_norm=self.q_norm, k_norm=self.k_norm,
@@ -243,12 +295,13 @@ class SinkAttention(Mixer):
         else:
             ops.rows_append(qkv, ctx.tok_pos, ctx.tok_row, cache.block_table, pages, **append)
         out = torch.empty((x.shape[0], H * dv), dtype=x.dtype, device=x.device)
-        params = make_params(ctx, q=qkv, q_stride=qkv.shape[1], q_head_stride=dk, out=out, cache=cache, H=H, KV=KV, dk=dk, dv=dv,
+        g_at = qkv.data_ptr() + ((H + KV) * dk + (0 if self.value_from_key else KV * dv)) * qkv.element_size()      # where a gate's columns begin
+        params = make_params(ctx, q=q, q_stride=q.shape[1], q_head_stride=dk, out=out, cache=cache, H=H, KV=KV, dk=dk, dv=dv,
                              row_width=dk + dv, k_off=0, v_off=dk, scale=self.scale, window=self.window, sink=self.sink,
-                             softcap=self.softcap, dist_bias=self.dist_table)
+                             softcap=self.softcap, dist_bias=self.dist_table, chunk=self.chunk, gate_ptr=g_at if self.head_gate else None,
+                             gate_stride=qkv.shape[1] if self.head_gate else 0)
         run(ctx, params)
         if self.has_gate:
-            g_at = qkv.data_ptr() + ((H + KV) * dk + (0 if self.value_from_key else KV * dv)) * qkv.element_size()
             ops.sigmoid_gate(out, g_at, qkv.shape[1], out)
         y = linear.linear(ctx, out, self.w_o, out_dtype=torch.float32 if self.wide_output else None)
         if self.out_bias is not None and not self.fold_out_bias:

@@ -64,6 +64,10 @@ Other workloads (``--workload``), each printing one JSON line of the same shape:
                head, windowed latent attention with a sink and an output gate, experts chosen in groups, identity experts)
                beside Yi, Mufalix, Pibalorn and Roletar, measured as the roletar workload is
 
+  burolorn     the Burolorn design (attention over chunks with a sink and a gate per head behind short convolutions, values mixed
+               across layers, token inputs from a second table, experts in groups ranked by two scores) beside Yi, Pibalorn,
+               Mevulix and Vazunex, measured as the roletar workload is
+
 ``--impl reference`` runs the unmodified hoenza/DELTA engine (baseline/reference_arm.py) on the
 default workload and prints its line.
 """
@@ -478,14 +482,28 @@ def vazunex_config(d: int) -> dict:
                 layers=[dict(L, mlp=mlp) for L in (ssd, delta, lat, delta, ssd, lat)])
 
 
+def burolorn_config(d: int) -> dict:
+    """A Burolorn model with layers of the sizes of a real model of width d: attention of d/128 heads of 128 on d/512 key-value heads behind
+    convolutions of 4 taps, 64 of 128 entries rotated, chunks of 1,024 tokens in two of three layers, values mixed across layers; token
+    inputs of 256; dense gated feed-forwards and mixtures of 16 experts (4 chosen, d/2 wide each, and a shared expert; 2 of 4 groups are
+    kept) take turns."""
+    H = d // 128
+    att = dict(heads=H, kv_heads=max(1, H // 4), dim=128, vdim=128, scale=0.09, conv=4, rot=dict(base=500000.0, dims=64), v_mix=True)
+    experts = dict(kind="moe", router=dict(experts=16, top=4, groups=dict(count=4, keep=2), scale=2.0), expert=dict(ff=d // 2), shared=dict(ff=d // 2))
+    dense = dict(kind="dense", ff=(8 * d // 3 + 255) // 256 * 256)
+    return dict(architecture="Burolorn", vocab=32000, width=d, norm=dict(eps=1e-5), logit_scale=0.5, token_side=dict(dim=256),
+                layers=[dict(type="attention", mixer=dict(att, mask=dict(size=1024)) if i % 3 < 2 else att, mlp=dense if i % 2 == 0 else experts)
+                        for i in range(6)])
+
+
 def roletar_workload(args) -> int:
     return design_workload(args, "roletar")
 
 
 def design_workload(args, design: str) -> int:
-    """Prefill (one prompt of 2,048 tokens in one step) and decode (batch 8 at context 2,048) of a design (Roletar, Pibalorn, Mufalix, Mevulix, Vazunex) beside the
+    """Prefill (one prompt of 2,048 tokens in one step) and decode (batch 8 at context 2,048) of a design (Roletar, Pibalorn, Mufalix, Mevulix, Vazunex, Burolorn) beside the
     Yi architecture at equal width and layer count (Mufalix also beside Pibalorn, the closest design; Mevulix beside Pibalorn and Roletar;
-    Vazunex beside Mufalix, Pibalorn and Roletar), through ``ModelRunner.step``, timed with CUDA events after warm-up with
+    Vazunex beside Mufalix, Pibalorn and Roletar; Burolorn beside Mevulix, Vazunex and Pibalorn), through ``ModelRunner.step``, timed with CUDA events after warm-up with
     the L2 flushed before every timed step; then every launcher's share of one such step, with the fraction of the measured
     peaks that the design's own kernels and their Yi counterparts reach."""
     import torch
@@ -566,11 +584,12 @@ def design_workload(args, design: str) -> int:
 
     launches = 0
     for d in args.width:
-        rc = {"roletar": roletar_config, "pibalorn": pibalorn_config, "mufalix": mufalix_config, "mevulix": mevulix_config, "vazunex": vazunex_config}[design](d)
+        rc = {"roletar": roletar_config, "pibalorn": pibalorn_config, "mufalix": mufalix_config, "mevulix": mevulix_config, "vazunex": vazunex_config,
+              "burolorn": burolorn_config}[design](d)
         runs = 6
         yc = yi_like_config(d, runs)
         a, b = measure(rc, rc["vocab"]), measure(yc, yc["vocab_size"])
-        if design in ("mufalix", "mevulix", "vazunex"):     # the closest design of the engine (32-bit stream, layer norms, experts beside a shared one) as well
+        if design in ("mufalix", "mevulix", "vazunex", "burolorn"):     # the closest design of the engine (32-bit stream, layer norms, experts beside a shared one) as well
             pc = pibalorn_config(d)
             c = measure(pc, pc["vocab"])
         if design in ("mevulix", "vazunex"):     # and the one whose mixers are the closest (latent attention, attention with a sink over a cache of rows)
@@ -579,6 +598,9 @@ def design_workload(args, design: str) -> int:
         if design == "vazunex":     # recurrent mixers behind a 32-bit stream, gated norms, a windowed attention with a sink and a gate
             mc = mufalix_config(d)
             c3 = measure(mc, mc["vocab"])
+        if design == "burolorn":     # attention with a sink, dense layers and mixtures in turn; short convolutions
+            ec, zc = mevulix_config(d), vazunex_config(d)
+            c4, c5 = measure(ec, ec["vocab"]), measure(zc, zc["vocab"])
         launches += a["launches_per_decode_step"]
         H = d // 128
         # what the kernels of one step have to move or compute, per launcher (prefill of T tokens unless said otherwise)
@@ -630,13 +652,14 @@ def design_workload(args, design: str) -> int:
             }
         if design == "mufalix":
             work = mufalix_work()
-        if design == "vazunex":
+
+        def vazunex_work():
             top, F, Hs, P, Ns, G, Wn = 4, d // 2, d // 32, 64, 128, 2, 1024
             n_ssd, n_delta, n_lat, n_moe = 2, 2, 2, 6
             ch = Hs * P + 2 * G * Ns                  # channels of a state-space layer's convolution
             seen = Wn * T - Wn * (Wn - 1) // 2
             real = 16 / 20                           # the share of the choices that are experts, when the choices are spread evenly
-            work = {
+            return {
                 "residual_norm": ((2 * d * 4 + 3 * d * 2) * T * (2 * runs), 0),
                 "embedding_pair": ((d * 2 + d * 4) * T, 0),
                 "conv_silu": ((2 * ch * n_ssd + 2 * 3 * d * n_delta) * 2 * T, 0),
@@ -652,11 +675,14 @@ def design_workload(args, design: str) -> int:
                 "gemm_nt_plain_batched": (0, 2 * T * H * (128 * 256 + 256 * 128) * n_lat),
                 "attention_rows_mma": (0, 2 * H * (320 + 256) * seen * n_lat),
             }
-        if design == "mevulix":
+        if design == "vazunex":
+            work = vazunex_work()
+
+        def mevulix_work():
             G, top, F, Fd, Rq = max(1, H // 4), 4, d // 2, (8 * d // 3 + 255) // 256 * 256, 3 * d // 8
             n_lat, n_att, n_own, n_moe, n_dense = 3, 3, 2, 4, 2      # latent layers, attention layers, of which with keys of their own, mixtures, dense
             pairs = T * (T + 1) // 2
-            work = {
+            return {
                 "sublayer_norm_add": ((2 * d * 4 + 2 * d * 2) * T * (2 * runs), 0),
                 "residual_norm": ((d * 4 + d * 2) * T, 0),
                 "rms_norm_strided": (2 * Rq * 2 * T * n_lat, 0),
@@ -670,6 +696,25 @@ def design_workload(args, design: str) -> int:
                 "library batched product": (0, 2 * T * H * (128 * 256 + 256 * 128) * n_lat),
                 "gemm_nt_plain_batched": (0, 2 * T * H * (128 * 256 + 256 * 128) * n_lat),
                 "attention_rows_mma": (0, 2 * H * (320 + 256) * pairs * n_lat + 4 * 128 * H * pairs * n_att),
+            }
+        if design == "mevulix":
+            work = mevulix_work()
+        if design == "burolorn":
+            G, top, F, Fd, n, Cn = max(1, H // 4), 4, d // 2, (8 * d // 3 + 255) // 256 * 256, 256, 1024
+            n_att, n_full, n_moe, n_dense = 6, 2, 3, 3
+            ch = (H + 2 * G) * 128                     # channels of a layer's convolutions
+            chunks = T // Cn * (Cn * (Cn + 1) // 2)      # (query, key) pairs inside the chunks
+            work = {
+                # per layer: two sums with a norm behind them (one of a sublayer's output, one of the token input), one that leaves the stream rounded
+                "residual_norm": ((3 * (2 * d * 4 + 2 * d * 2)) * T * runs, 0),
+                "embedding_pair": ((d * 2 + d * 4) * T, 0),
+                "rows_conv_append": ((2 * ch + G * 128) * 2 * T * n_att, 0),      # in, out, and the values that are mixed
+                "table_gate": (3 * n * 2 * T * runs, 0),
+                "glu_clamped": (3 * (Fd * n_dense + F * n_moe) * 2 * T, 0),
+                "experts_gather": (2 * top * d * 2 * T * n_moe, 0),
+                "experts_combine": ((top * d * 4 + 2 * d * 2) * T * n_moe, 0),
+                "experts_gemm_tc": (0, 2 * T * top * 3 * d * F * n_moe),
+                "attention_rows_mma": (0, 4 * 128 * H * (chunks * (n_att - n_full) + T * (T + 1) // 2 * n_full)),
             }
         roletar_work = {
             "stream_norm": ((2 * S * d * 4 + 2 * d * 2) * T * (2 * runs), 0),
@@ -715,7 +760,7 @@ def design_workload(args, design: str) -> int:
                              "decode_ms": c["decode_ms"], "decode_graph_ms": c["decode_graph_ms"],
                              "launches_per_decode_step": c["launches_per_decode_step"],
                              "prefill_launchers": fractions(c["prefill_launchers"], pibalorn_work()),
-                             "decode_launchers": fractions(c["decode_launchers"], {})}} if design in ("mufalix", "mevulix", "vazunex") else {}),
+                             "decode_launchers": fractions(c["decode_launchers"], {})}} if design in ("mufalix", "mevulix", "vazunex", "burolorn") else {}),
             **({"mufalix": {"prefill_tok_s": T / c3["prefill_ms"] * 1e3, "prefill_ms": c3["prefill_ms"], "decode_tok_s": B / c3["decode_ms"] * 1e3,
                             "decode_ms": c3["decode_ms"], "decode_graph_ms": c3["decode_graph_ms"],
                             "launches_per_decode_step": c3["launches_per_decode_step"],
@@ -726,6 +771,10 @@ def design_workload(args, design: str) -> int:
                             "launches_per_decode_step": c2["launches_per_decode_step"],
                             "prefill_launchers": fractions(c2["prefill_launchers"], roletar_work),
                             "decode_launchers": fractions(c2["decode_launchers"], {})}} if design in ("mevulix", "vazunex") else {}),
+            **({name: {"prefill_tok_s": T / m["prefill_ms"] * 1e3, "prefill_ms": m["prefill_ms"], "decode_tok_s": B / m["decode_ms"] * 1e3,
+                       "decode_ms": m["decode_ms"], "decode_graph_ms": m["decode_graph_ms"], "launches_per_decode_step": m["launches_per_decode_step"],
+                       "prefill_launchers": fractions(m["prefill_launchers"], table), "decode_launchers": fractions(m["decode_launchers"], {})}
+                for name, m, table in (("mevulix", c4, mevulix_work()), ("vazunex", c5, vazunex_work()))} if design == "burolorn" else {}),
             "config": {"width": d, "layer_runs": runs, "prefill_tokens": T, "decode_batch": B, "decode_context": CTX,
                        "l2": "flushed before every timed step"}}
     first = out["sizes"][str(args.width[0])]
@@ -751,9 +800,9 @@ def main() -> int:
     ap.add_argument("--enable_selective_cache", action="store_true", help="DELTA on (not the default run)")
     ap.add_argument("--full_cache_layers", nargs="+", type=int, default=[0, 1, 2, 14, 22])
     ap.add_argument("--subset_cache_size", type=int, default=64)
-    ap.add_argument("--workload", choices=["decode", "baseline", "yi9b-long", "yi34b-mixed", "grown", "long-prompt", "roletar", "pibalorn", "mufalix", "mevulix", "vazunex"],
+    ap.add_argument("--workload", choices=["decode", "baseline", "yi9b-long", "yi34b-mixed", "grown", "long-prompt", "roletar", "pibalorn", "mufalix", "mevulix", "vazunex", "burolorn"],
                     default="decode")
-    ap.add_argument("--width", type=int, nargs="+", default=[2048, 4096], help="--workload roletar / pibalorn / mufalix / mevulix / vazunex: the model widths that are measured")
+    ap.add_argument("--width", type=int, nargs="+", default=[2048, 4096], help="--workload roletar / pibalorn / mufalix / mevulix / vazunex / burolorn: the model widths that are measured")
     ap.add_argument("--generate", type=int, default=None, help="tokens generated per request in the other workloads (default: what the workload names)")
     args = ap.parse_args()
     if args.impl == "reference":
@@ -763,7 +812,7 @@ def main() -> int:
         return 2
     if args.warmup < 3:
         args.warmup = 3
-    if args.workload in ("roletar", "pibalorn", "mufalix", "mevulix", "vazunex"):
+    if args.workload in ("roletar", "pibalorn", "mufalix", "mevulix", "vazunex", "burolorn"):
         return design_workload(args, args.workload)
     if args.workload != "decode":
         return other_workload(args)

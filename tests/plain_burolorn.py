@@ -103,7 +103,9 @@ def attention(h, W, p, m, eps, first_values):
     layer mixes nothing."""
     T = h.shape[0]
     H, G, dk, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-    q, k, v = (rnd(causal_conv(lin(h, W[p + n]), W[p + n + ".conv"])) for n in "qkv")
+    q, k, v = (lin(h, W[p + n]) for n in "qkv")
+    if m.get("conv"):
+        q, k, v = (rnd(causal_conv(u, W[p + n + ".conv"])) for n, u in zip("qkv", (q, k, v)))
     q = rms_norm(q.view(T, H, dk), W[p + "q.norm"], eps)
     k = rms_norm(k.view(T, G, dk), W[p + "k.norm"], eps)
     pos = torch.arange(T)

@@ -35,7 +35,7 @@ class Ctx:
         return self._scratch[key][:n].view(*shape)
 
 
-def reference(rows, H, KV, dk, dv, scale, window, sink, latent):
+def reference(rows, H, KV, dk, dv, scale, window, sink, latent, chunk=None, gates=None):
     out = []
     for (before, n, Q, K, V) in rows:
         Q, K, V = Q.double(), K.double(), V.double()
@@ -43,6 +43,7 @@ def reference(rows, H, KV, dk, dv, scale, window, sink, latent):
         for i in range(n):
             pos = before + i
             lo = max(0, pos - window + 1) if window else 0
+            lo = max(lo, pos // chunk * chunk) if chunk else lo
             for h in range(H):
                 g = h // (H // KV)
                 s = (K[lo:pos + 1, g] @ Q[i, h]) * scale
@@ -51,10 +52,12 @@ def reference(rows, H, KV, dk, dv, scale, window, sink, latent):
                 den = e.sum() + (torch.exp(sink[h].double() - m) if sink is not None else 0.0)
                 o[i, h] = (e / den) @ V[lo:pos + 1, g]
         out.append(o)
-    return torch.cat(out)
+    o = torch.cat(out)
+    return o if gates is None else o * torch.sigmoid(gates.double())[:, :, None]
 
 
-def run_case(dtype, plain, shape, row_lens, window=None, use_sink=False, latent=False, spikes=(), seed=0, ps=16):
+def run_case(dtype, plain, shape, row_lens, window=None, use_sink=False, latent=False, spikes=(), seed=0, ps=16, chunk=None,
+             gated=False):
     """``row_lens``: (tokens cached before the step, new tokens) per batch row.  ``spikes``: (row, query index, key
     position): that query and that key get a large common component."""
     from delta_b200.kernels import ops
@@ -78,7 +81,8 @@ def run_case(dtype, plain, shape, row_lens, window=None, use_sink=False, latent=
         rows.append((before, n, Q, K, V))
     scale = 1.0 / math.sqrt(dk)
     sink = (torch.randn(H, generator=g) * 1.5) if use_sink else None
-    want = reference(rows, H, KV, dk, dv, scale, window, sink, latent)
+    gates = torch.randn(sum(n for _, n in row_lens), H + 5, generator=g).to(dt) if gated else None      # a head's gate is read in rows with more in them
+    want = reference(rows, H, KV, dk, dv, scale, window, sink, latent, chunk, gates[:, :H] if gated else None)
     # the cache, pages handed out in a shuffled order
     row_width = dk if latent else dk + dv
     k_off, v_off = 0, (0 if latent else dk)
@@ -111,8 +115,10 @@ def run_case(dtype, plain, shape, row_lens, window=None, use_sink=False, latent=
     # (the parameters hold raw addresses: every device tensor stays referenced until the result is read)
     dev = dict(cache=cache.cuda(), block_table=bt.cuda(), row_q_start=torch.tensor(starts, **i32), row_q_len=torch.tensor(q_lens, **i32),
                row_pos_start=torch.tensor([b for b, _ in row_lens], **i32), sink=sink.cuda() if sink is not None else None)
+    gates = gates.cuda() if gated else None
     params = ops.row_attn_params(q=q, q_stride=H * dk, q_head_stride=dk, out=out, tok_row=tok_row, tok_pos=tok_pos, H=H, KV=KV, dk=dk,
-                                 dv=dv, ps=ps, row_width=row_width, k_off=k_off, v_off=v_off, scale=scale, window=window or 0, err=err,
+                                 dv=dv, ps=ps, row_width=row_width, k_off=k_off, v_off=v_off, scale=scale, window=window or 0, chunk=chunk or 0, err=err,
+                                 gate_ptr=gates.data_ptr() if gated else None, gate_stride=H + 5,
                                  **dev)
     ctx.err = err
     row_attention.run(ctx, params)
@@ -159,3 +165,25 @@ def test_one_key_that_matters(dtype, plain):
             if kp < 0:
                 continue
             run_case(dtype, plain, shape, [(before, n), (5, 3)], window=W, use_sink=True, spikes=[(0, qi, kp)], seed=pos)
+
+
+@pytest.mark.parametrize("dtype,plain", KERNELS)
+@pytest.mark.parametrize("shape", [(6, 2, 64, 32), (8, 2, 128, 64), (4, 1, 48, 96), (2, 1, 96, 208), (32, 1, 64, 64)])
+def test_chunks_and_gates_of_heads(dtype, plain, shape):
+    """Chunks that end inside tiles of queries and of keys, beside a gate per head: portions, single tokens (their keys split over several
+    blocks), and both in one step."""
+    for chunk in (1, 7, 40, 64, 130):
+        run_case(dtype, plain, shape, [(0, 70), (33, 1), (0, 2), (100, 37), (15, 1), (129, 3)], use_sink=True, seed=1, chunk=chunk, gated=True)
+        run_case(dtype, plain, shape, [(130, 1), (0, 1), (39, 1), (40, 1)], use_sink=True, seed=2, chunk=chunk, gated=True)
+    run_case(dtype, plain, shape, [(0, 150), (500, 1)], seed=3, ps=8, gated=True)
+    run_case(dtype, plain, shape, [(700, 1), (640, 1)], seed=3, chunk=600, gated=True)
+
+
+@pytest.mark.parametrize("dtype,plain", KERNELS)
+def test_the_chunks_first_key_and_the_one_before(dtype, plain):
+    shape, C = (6, 2, 64, 32), 40
+    for before, n, qi in ((60, 50, 19), (79, 1, 0), (0, 130, 79), (0, 130, 80), (40, 1, 0), (41, 5, 3), (599, 1, 0)):
+        pos = before + qi
+        for kp in (pos // C * C, pos // C * C - 1, pos):
+            if kp >= 0:
+                run_case(dtype, plain, shape, [(before, n), (5, 3)], chunk=C, use_sink=True, spikes=[(0, qi, kp)], seed=pos)

@@ -62,6 +62,8 @@ _SIGNATURES = {
     "dk_latent_prepare": [P, I, P, P, P, I, P, I, P, I, I, I, P, F, P, I, I, I, I, I, I, P, I, I, P, P],
     "dk_attention_rows_mma_supported": [C.POINTER(RowAttnParams)],
     "dk_attention_rows_mma": [C.POINTER(RowAttnParams), I, I, P, P],
+    "dk_attention_rows_tc_supported": [C.POINTER(RowAttnParams)],
+    "dk_attention_rows_tc": [C.POINTER(RowAttnParams), I, P],
     "dk_gemm_nt_plain_batched": [P, P, P, I, I, I, I, I, I, I, L, L, L, I, I, P],
     "dk_embedding": [P, P, P, I, I, I, I, P, P],
     "dk_rms_norm": [P, P, P, P, P, I, I, F, I, I, I, P],

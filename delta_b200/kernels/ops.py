@@ -629,6 +629,17 @@ def attention_rows_mma(params: RowAttnParams, max_m: int, splits: int = 1, scrat
                                              _stream()), "attention_rows_mma", 2 if splits > 1 else 1)
 
 
+def attention_rows_tc_supported(params: RowAttnParams) -> bool:
+    """True when the tcgen05 kernel of the family takes these sizes (bfloat16; key and value sizes multiples of 8 from 64 to 128; no shaped
+    scores)."""
+    return bool(_l.load().dk_attention_rows_tc_supported(C.byref(params)))
+
+
+def attention_rows_tc(params: RowAttnParams, max_q_len: int):
+    """``max_q_len``: the most tokens any batch row brings among those that ``params.row_filter`` lets through."""
+    _l.check(_l.load().dk_attention_rows_tc(C.byref(params), int(max_q_len), _stream()), "attention_rows_tc")
+
+
 def rows_append_unit(src, tok_pos, tok_row, block_table, cache, *, H, KV, dk, dv, ps, row_width, k_off, v_off, table=None,
                      rot_dims=0, interleaved=True, unit_eps=None, value_from_key=False, bias=None, q_norm=None, k_norm=None,
                      pre_eps=0.0, norm_whole=False, q_temp=None, err=None):

@@ -56,6 +56,7 @@ from .base import MIXERS, PAGE, POSITION_ENCODINGS, CacheSpec, Mixer, PartSpec, 
 
 MAX_SPLITS = 32
 SINGLE_WARP_BLOCKS_PER_SM = 6      # blocks of one warp (a tile of a single token's heads) that an SM holds at a time
+TC_MIN_TOKENS = 64      # from this many tokens in some row, portions go to the tcgen05 kernel
 PARTIALS = "row_attention.partials"
 CONV_STATE = "conv"
 FIRST_VALUES = "row_attention.first_values."
@@ -77,17 +78,22 @@ def decode_splits(rows: int, kv_heads: int, group: int, max_keys: int, sm_count:
 
 def run(ctx, params) -> None:
     """Runs attention over a cache of rows with the kernels that fit the batch.  bfloat16 with key and value sizes that
-    are multiples of 16 goes to the tensor-core kernel: rows that bring several tokens in tiles of 64 query rows, rows
+    are multiples of 16 goes to the tensor cores: rows that bring several tokens to the tcgen05 kernel in tiles of 128 queries of a head
+    (``TC_MIN_TOKENS`` or more in some row, and sizes it takes), else to the warp-level kernel in tiles of 64 or 128 query rows; rows
     that bring one token as a tile of their group's heads with the keys split over several blocks; a mixed step
-    launches it once for each kind.  32 bit and other sizes go to the plain kernel.  In a replayable step nothing is
+    launches once for each kind.  32 bit and other sizes go to the plain kernel.  In a replayable step nothing is
     chosen from the step's host data."""
-    if plain(ctx) or not ops.attention_rows_mma_supported(params):
-        params.row_filter = 0
-        ops.attention_rows_plain(params)
-        return
-    group = params.H // params.KV
     singles = ctx.decode_only or any(n == 1 for n in ctx.host["q_lens"])
     several = not ctx.decode_only
+    tc = several and not plain(ctx) and ctx.max_q_len >= TC_MIN_TOKENS and ops.attention_rows_tc_supported(params)
+    if plain(ctx) or not ops.attention_rows_mma_supported(params):
+        params.row_filter = 0
+        if tc and not singles:
+            ops.attention_rows_tc(params, ctx.max_q_len)
+        else:
+            ops.attention_rows_plain(params)
+        return
+    group = params.H // params.KV
     if singles:
         params.row_filter = 1 if several else 0
         splits, scratch = 1, None
@@ -105,6 +111,9 @@ def run(ctx, params) -> None:
         ops.attention_rows_mma(params, group, splits, scratch)
     if several:
         params.row_filter = 2 if singles else 0
+        if tc:
+            ops.attention_rows_tc(params, ctx.max_q_len)
+            return
         ops.attention_rows_mma(params, ctx.max_q_len * group, 1, None)
 
 

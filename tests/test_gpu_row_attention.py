@@ -102,6 +102,10 @@ def run_case(dtype, plain, shape, row_lens, window=None, use_sink=False, latent=
             cache[page, :, off, k_off:k_off + dk] = K[j].to(dt)
             if not latent:
                 cache[page, :, off, v_off:v_off + dv] = V[j].to(dt)
+    for r, (before, _) in enumerate(row_lens):      # pages that no query of the step sees were given back
+        lo = max(0, before - window + 1) if window else 0
+        lo = max(lo, before // chunk * chunk) if chunk else lo
+        bt[r, :lo // ps] = -1
     q = torch.cat([Q.reshape(n, H * dk) for (_, n, Q, _, _) in rows]).to(dt).cuda()
     q_lens = [n for _, n in row_lens]
     starts = [sum(q_lens[:i]) for i in range(len(q_lens))]
@@ -187,3 +191,64 @@ def test_the_chunks_first_key_and_the_one_before(dtype, plain):
         for kp in (pos // C * C, pos // C * C - 1, pos):
             if kp >= 0:
                 run_case(dtype, plain, shape, [(before, n), (5, 3)], chunk=C, use_sink=True, spikes=[(0, qi, kp)], seed=pos)
+
+
+# ---- the tcgen05 kernel, also for portions shorter than those it is meant for ---------------------------------------------------
+
+TC_SHAPES = [(4, 2, 128, 128), (8, 2, 128, 64), (2, 1, 64, 128), (4, 4, 64, 64), (3, 1, 96, 80), (2, 1, 72, 104), (6, 3, 112, 64)]
+
+
+@pytest.fixture
+def tc_everywhere(monkeypatch):
+    from delta_b200.kernels import ops
+    from delta_b200.parts import row_attention
+    monkeypatch.setattr(row_attention, "TC_MIN_TOKENS", 2)
+    calls = []
+    real = ops.attention_rows_tc
+
+    def counted(*a):
+        calls.append(1)
+        return real(*a)
+    monkeypatch.setattr(ops, "attention_rows_tc", counted)
+    yield calls
+    assert calls, "the tcgen05 kernel did not run"
+
+
+@pytest.mark.parametrize("shape", TC_SHAPES)
+def test_tcgen05_portions(tc_everywhere, shape):
+    """One tile and many, rows of unequal lengths, contexts before them, windows and chunks that end inside tiles, sinks, gates, pages in runs
+    and scattered, pages of several sizes."""
+    for ps in ((16, 8, 64) if shape == TC_SHAPES[1] else (16,)):
+        run_case("bfloat16", False, shape, [(0, 70), (33, 40), (0, 2), (100, 37), (15, 9)], seed=1, ps=ps)
+        run_case("bfloat16", False, shape, [(0, 300), (130, 131)], use_sink=True, gated=True, seed=2, ps=ps)
+        run_case("bfloat16", False, shape, [(500, 260), (3, 128)], use_sink=True, window=200, seed=3, ps=ps)
+        run_case("bfloat16", False, shape, [(500, 260), (3, 128)], window=33, gated=True, seed=4, ps=ps)
+        for chunk in (1, 7, 100, 128, 300):
+            run_case("bfloat16", False, shape, [(0, 270), (290, 140), (129, 3)], use_sink=True, gated=True, chunk=chunk, seed=5, ps=ps)
+
+
+def test_tcgen05_beside_single_tokens(tc_everywhere):
+    run_case("bfloat16", False, (8, 2, 128, 64), [(700, 1), (0, 150), (31, 1), (200, 90), (0, 1), (40, 2)], use_sink=True, gated=True, chunk=120, seed=6)
+    run_case("bfloat16", False, (8, 2, 128, 128), [(0, 1), (700, 1), (600, 150)], seed=7)
+
+
+def test_tcgen05_many_pieces(tc_everywhere):
+    """More pieces of work than there are multiprocessors: a block takes several, of one tile and of many, one after the other."""
+    run_case("bfloat16", False, (16, 4, 128, 64), [(0, 900), (0, 20), (300, 700), (64, 128)], use_sink=True, gated=True, chunk=260, seed=8)
+    run_case("bfloat16", False, (16, 4, 64, 128), [(0, 900), (0, 20), (300, 700), (64, 128)], use_sink=True, seed=9)
+
+
+@pytest.mark.parametrize("kp", [0, 1, 15, 16, 47, 48, 127, 128, 200, 298])
+def test_tcgen05_one_key_that_matters(tc_everywhere, kp):
+    run_case("bfloat16", False, (4, 2, 128, 64), [(150, 150)], spikes=[(0, 149, kp)], seed=kp)
+
+
+@pytest.mark.parametrize("before,n,qi", [(60, 50, 19), (0, 130, 79), (0, 130, 80), (41, 5, 3), (119, 128, 0), (120, 128, 127), (0, 128, 40), (0, 128, 39)])
+def test_tcgen05_edges_of_chunks_and_windows(tc_everywhere, before, n, qi):
+    W, pos = 40, before + qi
+    for kp in (pos // W * W, pos // W * W - 1, pos):
+        if kp >= 0:
+            run_case("bfloat16", False, (4, 2, 128, 64), [(before, n), (5, 3)], chunk=W, use_sink=True, spikes=[(0, qi, kp)], seed=pos)
+    for kp in (pos - W + 1, pos - W):
+        if kp >= 0:
+            run_case("bfloat16", False, (4, 2, 64, 128), [(before, n), (5, 3)], window=W, use_sink=True, spikes=[(0, qi, kp)], seed=pos)

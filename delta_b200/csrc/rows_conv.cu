@@ -19,6 +19,7 @@ extern "C" int dk_conv_state(const void* xin, int in_stride, float* conv_state, 
 namespace {
 constexpr int WARPS = 4;          // units of a block
 constexpr int TILE = 8;           // tokens a warp takes in turn on prompt portions (inputs stay in registers between them)
+constexpr int VEC_TILE = 4;       // and side by side in the form for heads of 64 or 128
 constexpr int MAX_TAPS = 16;
 
 struct RowsConv {
@@ -288,6 +289,206 @@ __global__ void __launch_bounds__(WARPS * 32) rows_conv_pairs_kernel(const RowsC
   }
 }
 
+// bfloat16, 2 to 4 taps, heads of 32 VEC entries: a lane holds VEC entries that follow one another, and a warp takes TILE tokens of a row
+// with every load under way before the first sum is needed; the rotation's partner entries come from another lane.  The inputs
+// of earlier steps are bfloat16 values kept in 32 bit, so they are packed again without a loss.
+template <int VEC>
+struct Raw {
+  uint32_t r[VEC / 2];
+};
+template <int VEC>
+__device__ __forceinline__ Raw<VEC> load_raw(const __nv_bfloat16* p) {
+  Raw<VEC> v;
+  if constexpr (VEC == 2) v.r[0] = *reinterpret_cast<const uint32_t*>(p);
+  else {
+    const uint2 a = *reinterpret_cast<const uint2*>(p);
+    v.r[0] = a.x;
+    v.r[1] = a.y;
+  }
+  return v;
+}
+template <int VEC>
+__device__ __forceinline__ void store_raw(__nv_bfloat16* p, const float (&v)[VEC]) {
+  uint32_t r[VEC / 2];
+#pragma unroll
+  for (int e = 0; e < VEC / 2; ++e) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(v[2 * e], v[2 * e + 1]);
+    r[e] = *reinterpret_cast<const uint32_t*>(&h);
+  }
+  if constexpr (VEC == 2) *reinterpret_cast<uint32_t*>(p) = r[0];
+  else *reinterpret_cast<uint2*>(p) = make_uint2(r[0], r[1]);
+}
+template <int VEC>
+__device__ __forceinline__ void load_floats(const float* p, float (&v)[VEC]) {
+  if constexpr (VEC == 2) {
+    const float2 a = *reinterpret_cast<const float2*>(p);
+    v[0] = a.x; v[1] = a.y;
+  } else {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+  }
+}
+template <int VEC>
+__device__ __forceinline__ void unpack(const Raw<VEC>& raw, float (&v)[VEC]) {
+#pragma unroll
+  for (int e = 0; e < VEC / 2; ++e) {
+    v[2 * e] = __uint_as_float(raw.r[e] << 16);
+    v[2 * e + 1] = __uint_as_float(raw.r[e] & 0xffff0000u);
+  }
+}
+
+// The n <= TILE tokens from t0 on, all of batch row `row`.
+template <int TAPS, int VEC, int TILE>
+__device__ __forceinline__ void conv_tile(const RowsConv& p, const Unit& un, int t0, int n, int row, int lane) {
+  using bf16 = __nv_bfloat16;
+  const int i = lane * VEC;
+  const bf16* src = reinterpret_cast<const bf16*>(p.src) + un.c0 + i;
+  const int q0 = p.row_q_start[row], pos0 = p.tok_pos[t0];
+  float* st = p.conv_state + (size_t)p.row_slot[row] * (TAPS - 1) * p.C + un.c0 + i;
+  Raw<VEC> raw[TILE + TAPS - 1];
+#pragma unroll
+  for (int k = 0; k < TILE; ++k)
+    if (k < n) raw[TAPS - 1 + k] = load_raw<VEC>(src + (size_t)(t0 + k) * p.src_stride);
+#pragma unroll
+  for (int k = 0; k < TAPS - 1; ++k) {
+    const int at = t0 - q0 - (TAPS - 1) + k;      // index among the row's tokens of this step; negative: before it
+    if (at >= 0) {
+      raw[k] = load_raw<VEC>(src + (size_t)(q0 + at) * p.src_stride);
+    } else {
+      float v[VEC];
+      load_floats<VEC>(st + (size_t)(TAPS - 1 + at) * p.C, v);
+#pragma unroll
+      for (int e = 0; e < VEC / 2; ++e) {
+        const __nv_bfloat162 h = __floats2bfloat162_rn(v[2 * e], v[2 * e + 1]);
+        raw[k].r[e] = *reinterpret_cast<const uint32_t*>(&h);
+      }
+    }
+  }
+  float w[TAPS][VEC], nw[VEC];
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) load_floats<VEC>(p.w + (size_t)j * p.C + un.c0 + i, w[j]);
+  const float* norm = un.kind == 0 ? p.q_norm : (un.kind == 1 ? p.k_norm : nullptr);
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) nw[e] = 1.f;
+  if (norm != nullptr) load_floats<VEC>(norm + i, nw);
+  float a[TILE][VEC], ss[TILE];
+#pragma unroll
+  for (int k = 0; k < TILE; ++k) {
+    ss[k] = 0.f;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) a[k][e] = 0.f;
+    if (k < n) {
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        float v[VEC];
+        unpack<VEC>(raw[k + j], v);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) a[k][e] = fmaf(w[j][e], v[e], a[k][e]);
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss[k] += a[k][e] * a[k][e];
+    }
+  }
+  if (TILE == 1 && p.single) {      // the last TAPS - 1 inputs, this one included
+#pragma unroll
+    for (int j = 0; j < TAPS - 1; ++j) {
+      float v[VEC];
+      unpack<VEC>(raw[j + 1], v);
+#pragma unroll
+      for (int e = 0; e < VEC; e += 2) *reinterpret_cast<float2*>(st + (size_t)j * p.C + e) = make_float2(v[e], v[e + 1]);
+    }
+  }
+  if (un.kind == 2) {
+#pragma unroll
+    for (int k = 0; k < TILE; ++k) {
+      if (k >= n || !good_position(p, t0 + k, pos0 + k, lane)) continue;
+      bf16* first = p.mix_mode ? reinterpret_cast<bf16*>(p.first) + ((size_t)(t0 + k) * p.KV + un.head) * p.dv + i : nullptr;
+      if (p.mix_mode == 1) store_raw<VEC>(first, a[k]);
+      if (p.mix_mode == 2) {
+        float f[VEC];
+        unpack<VEC>(load_raw<VEC>(first), f);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) a[k][e] = (1.f - p.lambda) * a[k][e] + p.lambda * f[e];
+      }
+      bf16* crow = cache_row<bf16>(p, t0 + k, pos0 + k, row, un.head, lane);
+      if (crow != nullptr) store_raw<VEC>(crow + p.v_off + i, a[k]);
+    }
+    return;
+  }
+  if (norm != nullptr) {
+#pragma unroll
+    for (int k = 0; k < TILE; ++k) {
+      const float inv = rsqrtf(warp_sum(ss[k]) * (1.f / (32 * VEC)) + p.eps);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) a[k][e] *= inv * nw[e];
+    }
+  }
+  const int half = p.rot_dims / 2;
+  const bool turned = p.table != nullptr && i < p.rot_dims, front = i < half;
+  const int partner = turned ? (front ? lane + half / VEC : lane - half / VEC) : lane;
+  const int j0 = front ? i : i - half;
+#pragma unroll
+  for (int k = 0; k < TILE; ++k) {
+    if (k >= n) continue;
+    const int pos = pos0 + k;
+    const bool good = good_position(p, t0 + k, pos, lane);
+    if (p.table != nullptr) {
+      float o[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) o[e] = __shfl_sync(0xffffffffu, a[k][e], partner);
+      if (turned && good) {
+        const float* cs = p.table + (size_t)pos * p.rot_dims + 2 * j0;
+#pragma unroll
+        for (int e = 0; e < VEC; e += 2) {
+          const float4 t = *reinterpret_cast<const float4*>(cs + 2 * e);      // cos, sin of two pairs
+          a[k][e] = front ? a[k][e] * t.x - o[e] * t.y : a[k][e] * t.x + o[e] * t.y;
+          a[k][e + 1] = front ? a[k][e + 1] * t.z - o[e + 1] * t.w : a[k][e + 1] * t.z + o[e + 1] * t.w;
+        }
+      }
+    }
+    if (!good) continue;
+    if (un.kind == 0) {
+      store_raw<VEC>(reinterpret_cast<bf16*>(p.q_out) + ((size_t)(t0 + k) * p.H + un.head) * p.dk + i, a[k]);
+    } else {
+      bf16* crow = cache_row<bf16>(p, t0 + k, pos, row, un.head, lane);
+      if (crow != nullptr) store_raw<VEC>(crow + p.k_off + i, a[k]);
+    }
+  }
+}
+
+template <int TAPS, int VK, int VV, int TILE>
+__global__ void __launch_bounds__(WARPS * 32) rows_conv_vec_kernel(const RowsConv p) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int u = blockIdx.y * WARPS + warp;
+  if (u >= p.H + 2 * p.KV) return;
+  const Unit un = unit_of(p, u);
+  const int t0 = blockIdx.x * TILE, n = min(TILE, p.T - t0);
+  const int row = p.tok_row[t0];
+  if (TILE == 1 || p.tok_row[t0 + n - 1] == row) {
+    if (un.kind == 2) conv_tile<TAPS, VV, TILE>(p, un, t0, n, row, lane);
+    else conv_tile<TAPS, VK, TILE>(p, un, t0, n, row, lane);
+  } else {      // the tile's tokens belong to several rows
+    for (int k = 0; k < n; ++k) {
+      if (un.kind == 2) conv_tile<TAPS, VV, 1>(p, un, t0 + k, 1, p.tok_row[t0 + k], lane);
+      else conv_tile<TAPS, VK, 1>(p, un, t0 + k, 1, p.tok_row[t0 + k], lane);
+    }
+  }
+}
+
+template <int TAPS, int TILE>
+void launch_vec(const RowsConv& p, dim3 grid, cudaStream_t stream) {
+  if (p.dk == 128 && p.dv == 128) rows_conv_vec_kernel<TAPS, 4, 4, TILE><<<grid, WARPS * 32, 0, stream>>>(p);
+  else if (p.dk == 128) rows_conv_vec_kernel<TAPS, 4, 2, TILE><<<grid, WARPS * 32, 0, stream>>>(p);
+  else if (p.dv == 128) rows_conv_vec_kernel<TAPS, 2, 4, TILE><<<grid, WARPS * 32, 0, stream>>>(p);
+  else rows_conv_vec_kernel<TAPS, 2, 2, TILE><<<grid, WARPS * 32, 0, stream>>>(p);
+}
+template <int TILE>
+void launch_vec_taps(const RowsConv& p, dim3 grid, cudaStream_t stream) {
+  if (p.taps == 2) launch_vec<2, TILE>(p, grid, stream);
+  else if (p.taps == 3) launch_vec<3, TILE>(p, grid, stream);
+  else launch_vec<4, TILE>(p, grid, stream);
+}
+
 template <typename T, int TAPS>
 void launch_pairs(const RowsConv& p, int np, int tile, dim3 grid, size_t smem, cudaStream_t stream) {
   if (np == 1) rows_conv_pairs_kernel<T, TAPS, 1><<<grid, WARPS * 32, smem, stream>>>(p, tile);
@@ -335,7 +536,17 @@ extern "C" int dk_rows_conv_append(const void* src, int src_stride, const float*
   const bool pairs = taps >= 2 && taps <= 4 && dk % 2 == 0 && dv % 2 == 0 && D <= 256 && src_stride % 2 == 0 && row_width % 2 == 0 && k_off % 2 == 0 &&
                      v_off % 2 == 0 && aligned(src, pair) && aligned(q_out, pair) && aligned(cache, pair) && aligned(first, pair) &&
                      aligned(w, 8) && aligned(conv_state, 8) && aligned(q_norm, 8) && aligned(k_norm, 8);
-  if (pairs) {
+  const int vk = dk / 32;
+  const bool vecs = pairs && dtype == DK_BF16 && (dk == 64 || dk == 128) && (dv == 64 || dv == 128) && src_stride % 4 == 0 && row_width % 4 == 0 &&
+                    k_off % 4 == 0 && v_off % 4 == 0 && aligned(src, 8) && aligned(q_out, 8) && aligned(cache, 8) && aligned(first, 8) && aligned(w, 16) &&
+                    aligned(conv_state, 16) && aligned(q_norm, 16) && aligned(k_norm, 16) && aligned(table, 16) &&
+                    (table == nullptr || (!interleaved && (rot_dims / 2) % vk == 0 && rot_dims % 4 == 0));
+  if (vecs) {
+    // few tokens: one a warp, so that the step has many warps; many: VEC_TILE side by side, so that most inputs are read once
+    const bool many = !single && (long long)T_ * units >= 16LL * VEC_TILE * dk_sm_count();
+    if (many) launch_vec_taps<VEC_TILE>(p, dim3((T_ + VEC_TILE - 1) / VEC_TILE, unit_blocks), stream);
+    else launch_vec_taps<1>(p, dim3(T_, unit_blocks), stream);
+  } else if (pairs) {
     const int np = D <= 64 ? 1 : (D <= 128 ? 2 : 4);
     // few tokens: one a warp, so that the step has many warps; many: TILE in turn, so that the inputs are read once
     const int tile = (long long)T_ * units >= 32LL * TILE * dk_sm_count() ? TILE : 1;

@@ -291,66 +291,78 @@ def step_rows(lens, slots, before):
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("taps", [0, 1, 2, 3, 4, 6])
 @pytest.mark.parametrize("H,KV,dk,dv,rot,interleaved", [(4, 2, 64, 32, 32, False), (3, 1, 128, 128, 128, False), (2, 2, 30, 66, 10, True),
-                                                        (2, 1, 200, 24, 64, False), (3, 3, 11, 7, 4, False), (1, 1, 2, 2, 0, False)])
+                                                        (2, 1, 200, 24, 64, False), (3, 3, 11, 7, 4, False), (1, 1, 2, 2, 0, False),
+                                                        (4, 2, 128, 64, 64, False), (2, 2, 64, 64, 8, False), (5, 1, 64, 128, 0, False)])
 def test_convolution_norm_rotation_and_append(dtype, taps, H, KV, dk, dv, rot, interleaved):
-    """From projected rows to queries and cache rows, with inputs of earlier steps in the state: the kernel that keeps pairs in registers and
+    """From projected rows to queries and cache rows, with inputs of earlier steps in the state: the kernels that keep heads in registers and
     the one for any size, rows of several tokens and steps of single ones, value mixing of every kind, shuffled pages; and the state that
     is left."""
+    for lens in ([1, 19, 2, 8], [1, 1, 1, 1]):
+        check_conv_append(dtype, taps, H, KV, dk, dv, rot, interleaved, lens, [9, 0, 30, 5])
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("taps,H,KV,dk,dv", [(4, 8, 2, 128, 64), (3, 8, 4, 64, 128), (2, 12, 2, 96, 32), (4, 8, 2, 64, 64), (4, 8, 2, 128, 128)])
+def test_convolution_over_long_portions(dtype, taps, H, KV, dk, dv):
+    """Enough tokens for the tiles of several tokens a warp, whose edges fall inside rows, between them and on rows of one or two tokens."""
+    check_conv_append(dtype, taps, H, KV, dk, dv, 32, False, [3, 1001, 1, 2, 1500], [0, 57, 9, 0, 700], ps=16)
+
+
+def check_conv_append(dtype, taps, H, KV, dk, dv, rot, interleaved, lens, before, ps=4):
     from delta_b200.kernels import ops
     g = torch.Generator().manual_seed(taps * 100 + dk)
-    ps, C = 4, (H + KV) * dk + KV * dv
+    C = (H + KV) * dk + KV * dv
     tol = 3e-6 if dtype == torch.float32 else 1e-2
-    for lens in ([1, 19, 2, 8], [1, 1, 1, 1]):
-        before, slots, T = [9, 0, 30, 5], [3, 0, 4, 1], sum(lens)
-        src = torch.randn(T, C + 6, generator=g).to(dtype)
-        w = torch.randn(max(taps, 1), C, generator=g)
-        state = torch.randn(5, max(taps - 1, 1), C, generator=g)
-        qn, kn = torch.rand(dk, generator=g) + 0.5, torch.rand(dk, generator=g) + 0.5
-        ang = torch.arange(64, dtype=plain.F)[:, None] * 50.0 ** (-2.0 * torch.arange(max(rot // 2, 1), dtype=plain.F) / max(rot, 2))[None]
-        table = torch.stack([torch.cos(ang), torch.sin(ang)], dim=-1).float()
-        rows, toks, starts = step_rows(lens, slots, before)
-        n_pages = 60
-        order = torch.randperm(n_pages, generator=g).tolist()
-        bt = torch.tensor([[order[10 * r + i] for i in range(10)] for r in range(4)], dtype=torch.int32)
-        first0 = torch.randn(T, KV * dv, generator=g).to(dtype)
-        for mix in (None, "first", 0.3):
-            for single in ((False, True) if max(lens) == 1 else (False,)):
-                st, cache = state.to(DEV).clone(), torch.zeros(n_pages, KV, ps, dk + dv, dtype=dtype, device=DEV)
-                q, first, err = torch.empty(T, H * dk, dtype=dtype, device=DEV), first0.to(DEV).clone(), ops.new_error_record(DEV)
-                dev = dict(src=src.to(DEV), w=w.to(DEV), bt=bt.to(DEV), qn=qn.to(DEV), kn=kn.to(DEV), table=table.to(DEV))
-                ops.rows_conv_append(dev["src"], q, dev["w"] if taps else None, st if taps > 1 else None, toks["tok_pos"], toks["tok_row"], dev["bt"], cache,
-                                     H=H, KV=KV, dk=dk, dv=dv, ps=ps, row_width=dk + dv, k_off=0, v_off=dk, table=dev["table"] if rot else None,
-                                     rot_dims=rot, interleaved=interleaved, q_norm=dev["qn"], k_norm=dev["kn"], eps=1e-5, first=first, mix=mix,
-                                     single=single, err=err, **rows)
-                ops.raise_if_error(err)
-                q, cache, first, st = q.cpu().double(), cache.cpu().double(), first.cpu().double(), st.cpu()
-                for r, n in enumerate(lens):
-                    x = src[starts[r]:starts[r] + n, :C].double()
-                    seq = torch.cat([state[slots[r]].double()[:max(taps - 1, 0)], x])
-                    u = sum(seq[j:j + n] * w[j].double() for j in range(taps)) if taps else x
-                    pos = torch.arange(before[r], before[r] + n)
-                    heads = []
-                    for part, weight in ((u[:, :H * dk].view(n, H, dk), qn), (u[:, H * dk:(H + KV) * dk].view(n, KV, dk), kn)):
-                        y = plain.rms_norm(part, weight, 1e-5)
-                        if rot:
-                            perm = [2 * i for i in range(rot // 2)] + [2 * i + 1 for i in range(rot // 2)] if interleaved else list(range(rot))
-                            y = y.clone()
-                            y[..., perm] = plain.rotate_halves(y[..., perm], pos, dict(base=50.0, dims=rot))
-                        heads.append(y)
-                    v = u[:, (H + KV) * dk:]
-                    f = first0[starts[r]:starts[r] + n].double()
-                    if mix == "first":
-                        assert (first[starts[r]:starts[r] + n] - v).abs().max().item() <= tol * v.abs().max().item()
-                    if isinstance(mix, float):
-                        v = plain.mixed_values(v, f, mix)
-                        assert torch.equal(first[starts[r]:starts[r] + n], f)
-                    got = torch.stack([torch.cat([cache[bt[r, p // ps], :, p % ps]], dim=0) for p in pos.tolist()])      # [n, KV, dk + dv]
-                    for a, b in ((q[starts[r]:starts[r] + n].view(n, H, dk), heads[0]), (got[..., :dk], heads[1]), (got[..., dk:], v.reshape(n, KV, dv))):
-                        assert (a - b).abs().max().item() <= tol * max(1.0, b.abs().max().item()), (r, mix, single)
-                    if taps > 1:
-                        assert torch.equal(st[slots[r]], seq[-(taps - 1):].float())
+    slots, T = [3, 0, 4, 1, 5][:len(lens)], sum(lens)
+    src = torch.randn(T, C + 8, generator=g).to(dtype)
+    w = torch.randn(max(taps, 1), C, generator=g)
+    state = torch.randn(7, max(taps - 1, 1), C, generator=g).to(dtype).float()      # (what a state holds are inputs as they were projected)
+    qn, kn = torch.rand(dk, generator=g) + 0.5, torch.rand(dk, generator=g) + 0.5
+    ang = torch.arange(max(b + n for b, n in zip(before, lens)), dtype=plain.F)[:, None] * 50.0 ** (-2.0 * torch.arange(max(rot // 2, 1), dtype=plain.F) / max(rot, 2))[None]
+    table = torch.stack([torch.cos(ang), torch.sin(ang)], dim=-1).float()
+    rows, toks, starts = step_rows(lens, slots, before)
+    per = max(-(-(b + n) // ps) for b, n in zip(before, lens))
+    n_pages = per * len(lens) + 3
+    bt = torch.randperm(n_pages, generator=g)[:per * len(lens)].view(len(lens), per).int()
+    first0 = torch.randn(T, KV * dv, generator=g).to(dtype)
+    for mix in (None, "first", 0.3):
+        for single in ((False, True) if max(lens) == 1 else (False,)):
+            st, cache = state.to(DEV).clone(), torch.zeros(n_pages, KV, ps, dk + dv, dtype=dtype, device=DEV)
+            q, first, err = torch.empty(T, H * dk, dtype=dtype, device=DEV), first0.to(DEV).clone(), ops.new_error_record(DEV)
+            dev = dict(src=src.to(DEV), w=w.to(DEV), bt=bt.to(DEV), qn=qn.to(DEV), kn=kn.to(DEV), table=table.to(DEV))
+            ops.rows_conv_append(dev["src"], q, dev["w"] if taps else None, st if taps > 1 else None, toks["tok_pos"], toks["tok_row"], dev["bt"], cache,
+                                 H=H, KV=KV, dk=dk, dv=dv, ps=ps, row_width=dk + dv, k_off=0, v_off=dk, table=dev["table"] if rot else None,
+                                 rot_dims=rot, interleaved=interleaved, q_norm=dev["qn"], k_norm=dev["kn"], eps=1e-5, first=first, mix=mix,
+                                 single=single, err=err, **rows)
+            ops.raise_if_error(err)
+            q, cache, first, st = q.cpu().double(), cache.cpu().double(), first.cpu().double(), st.cpu()
+            for r, n in enumerate(lens):
+                x = src[starts[r]:starts[r] + n, :C].double()
+                seq = torch.cat([state[slots[r]].double()[:max(taps - 1, 0)], x])
+                u = sum(seq[j:j + n] * w[j].double() for j in range(taps)) if taps else x
+                pos = torch.arange(before[r], before[r] + n)
+                heads = []
+                for part, weight in ((u[:, :H * dk].view(n, H, dk), qn), (u[:, H * dk:(H + KV) * dk].view(n, KV, dk), kn)):
+                    y = plain.rms_norm(part, weight, 1e-5)
+                    if rot:
+                        perm = [2 * i for i in range(rot // 2)] + [2 * i + 1 for i in range(rot // 2)] if interleaved else list(range(rot))
+                        y = y.clone()
+                        y[..., perm] = plain.rotate_halves(y[..., perm], pos, dict(base=50.0, dims=rot))
+                    heads.append(y)
+                v = u[:, (H + KV) * dk:]
+                f = first0[starts[r]:starts[r] + n].double()
+                if mix == "first":
+                    assert (first[starts[r]:starts[r] + n] - v).abs().max().item() <= tol * v.abs().max().item()
+                if isinstance(mix, float):
+                    v = plain.mixed_values(v, f, mix)
+                    assert torch.equal(first[starts[r]:starts[r] + n], f)
+                got = cache[bt[r].long()[pos // ps], :, pos % ps]      # [n, KV, dk + dv]
+                for a, b in ((q[starts[r]:starts[r] + n].view(n, H, dk), heads[0]), (got[..., :dk], heads[1]), (got[..., dk:], v.reshape(n, KV, dv))):
+                    assert (a - b).abs().max().item() <= tol * max(1.0, b.abs().max().item()), (r, mix, single)
                 if taps > 1:
-                    assert torch.equal(st[2], state[2])            # a slot of no row
+                    assert torch.equal(st[slots[r]], seq[-(taps - 1):].float())
+            if taps > 1:
+                assert torch.equal(st[2], state[2])            # a slot of no row
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])

@@ -72,24 +72,31 @@ __global__ void __launch_bounds__(WARPS * 32) attention_rows_mma_kernel(const Dk
     const __nv_bfloat16* src = q + (size_t)(q_start + m / G) * p.q_stride + (size_t)(g * G + m % G) * p.q_head_stride + part_c * 8;
     cp_async_16(smem_u32(q_smem + r * QS + ((part_c ^ (r & 7)) * 16)), src, true);
   }
+  // A tile of keys and values: every lane looks the pages of KT / 32 tokens up, then the warps take the tokens in turn, 8, 16 or 32 lanes
+  // a token by the row's width (the page size is a power of two).
+  const int ps_shift = 31 - __clz(ps);
+  const int lpt_shift = CPR > 16 ? 5 : (CPR > 8 ? 4 : 3);
+  const int sub = lane >> lpt_shift, chunk0 = lane & ((1 << lpt_shift) - 1), tpi = 32 >> lpt_shift;
   auto load_tile = [&](int kt, int stage) {
     unsigned char* dst = kv_smem + (size_t)stage * KT * ROWS;
-    for (int c = tid; c < KT * CPR; c += THREADS) {
-      const int tok = c / CPR, part_c = c % CPR;
-      const int key = kt * KT + tok;
-      bool valid = false;
-      size_t off = 0;
+#pragma unroll
+    for (int i = 0; i < KT / 32; ++i) {
+      const int key = kt * KT + i * 32 + lane;
+      int at = -1;      // the token's row of the cache
       if (key <= last_pos && key >= lo_tile) {
-        const int lp = key / ps;
+        const int lp = key >> ps_shift;
         const int page = lp < p.max_pages ? p.block_table[(size_t)row * p.max_pages + lp] : -1;
-        if (page < 0 || page >= p.num_pages) {
-          if (part_c == 0) dk_report(p.err, DK_DEV_BAD_PAGE, q_start, lp, page);
-        } else {
-          valid = true;
-          off = (((size_t)page * p.KV + g) * ps + key % ps) * p.row_width + part_c * 8;
-        }
+        if (page < 0 || page >= p.num_pages) dk_report(p.err, DK_DEV_BAD_PAGE, q_start, lp, page);
+        else at = ((page * p.KV + g) << ps_shift) + (key & (ps - 1));
       }
-      cp_async_16(smem_u32(dst + tok * ROWS + ((part_c ^ (tok & 7)) * 16)), cache + off, valid);
+#pragma unroll 4
+      for (int t = warp * tpi; t < 32; t += WARPS * tpi) {
+        const int tok = t + sub;
+        const int from = __shfl_sync(0xffffffffu, at, tok);
+        unsigned char* trow = dst + (i * 32 + tok) * ROWS;
+        const __nv_bfloat16* src = cache + (size_t)max(from, 0) * p.row_width;
+        for (int c = chunk0; c < CPR; c += 1 << lpt_shift) cp_async_16(smem_u32(trow + ((c ^ (tok & 7)) * 16)), src + c * 8, from >= 0);
+      }
     }
   };
 
@@ -310,29 +317,45 @@ __global__ void __launch_bounds__(WARPS * 32) attention_rows_mma_kernel(const Dk
 }
 
 // one block per (token of a single-token row, head): sums the splits' partial results
+constexpr int MERGE_SPLITS = 128;
 __global__ void attention_rows_merge_kernel(const DkRowAttnParams p, const float* __restrict__ part, int splits) {
+  __shared__ float factor[MERGE_SPLITS];      // what a split's sums are multiplied by
+  __shared__ float inv_sum;
   const int t = blockIdx.x, head = blockIdx.y;
   const int row = p.tok_row[t];
   const int q_len = p.row_q_len[row];
   if ((p.row_filter == 2 && q_len == 1) || (p.row_filter == 1 && q_len != 1)) return;
-  const int dv = p.dv;
+  const int dv = p.dv, lane = threadIdx.x;
   const float* src = part + ((size_t)t * p.H + head) * splits * (dv + 2);
-  float mf = p.sink != nullptr ? p.sink[head] * LOG2E : -INFINITY;
-  for (int s = 0; s < splits; ++s) mf = fmaxf(mf, src[(size_t)s * (dv + 2) + dv]);
-  float l = p.sink != nullptr ? exp2f(p.sink[head] * LOG2E - mf) : 0.f;
-  for (int s = 0; s < splits; ++s) {
-    const float ms = src[(size_t)s * (dv + 2) + dv];
-    if (ms != -INFINITY) l += src[(size_t)s * (dv + 2) + dv + 1] * exp2f(ms - mf);
+  if (threadIdx.x < 32) {
+    float m[MERGE_SPLITS / 32], l[MERGE_SPLITS / 32];
+    float mf = p.sink != nullptr ? p.sink[head] * LOG2E : -INFINITY;
+#pragma unroll
+    for (int i = 0; i < MERGE_SPLITS / 32; ++i) {
+      const int s = lane + 32 * i;
+      m[i] = s < splits ? src[(size_t)s * (dv + 2) + dv] : -INFINITY;
+      l[i] = s < splits ? src[(size_t)s * (dv + 2) + dv + 1] : 0.f;
+      mf = fmaxf(mf, m[i]);
+    }
+    mf = warp_max(mf);
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < MERGE_SPLITS / 32; ++i) {
+      const float f = m[i] == -INFINITY ? 0.f : exp2f(m[i] - mf);      // (a split whose keys are all masked has neither sum nor values)
+      factor[lane + 32 * i] = f;
+      if (m[i] != -INFINITY) sum += l[i] * f;
+    }
+    sum = warp_sum(sum);
+    if (p.sink != nullptr) sum += exp2f(p.sink[head] * LOG2E - mf);
+    if (lane == 0) inv_sum = sum > 0.f ? row_head_gate<__nv_bfloat16>(p, t, head) / sum : 0.f;
   }
-  const float inv = l > 0.f ? row_head_gate<__nv_bfloat16>(p, t, head) / l : 0.f;
+  __syncthreads();
   __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(p.out) + ((size_t)t * p.H + head) * dv;
   for (int d = threadIdx.x; d < dv; d += blockDim.x) {
     float a = 0.f;
-    for (int s = 0; s < splits; ++s) {
-      const float ms = src[(size_t)s * (dv + 2) + dv];
-      if (ms != -INFINITY) a = fmaf(src[(size_t)s * (dv + 2) + d], exp2f(ms - mf), a);
-    }
-    orow[d] = __float2bfloat16_rn(a * inv);
+#pragma unroll 8
+    for (int s = 0; s < splits; ++s) a = fmaf(src[(size_t)s * (dv + 2) + d], factor[s], a);
+    orow[d] = __float2bfloat16_rn(a * inv_sum);
   }
 }
 
@@ -388,12 +411,13 @@ extern "C" int dk_attention_rows_mma(const DkRowAttnParams* pp, int max_m, int s
   if (p.T == 0 || p.rows == 0) return 0;
   DK_REQUIRE(dk_attention_rows_mma_supported(pp), "attention_rows_mma: sizes not taken (bfloat16; key and value sizes multiples of 16, value "
              "at most 256; offsets and strides multiples of 8): dk=%d dv=%d width=%d", p.dk, p.dv, p.row_width);
-  DK_REQUIRE(max_m >= 1 && splits >= 1 && splits <= 65535, "attention_rows_mma: bad max_m %d or splits %d", max_m, splits);
+  DK_REQUIRE(max_m >= 1 && splits >= 1 && splits <= MERGE_SPLITS, "attention_rows_mma: bad max_m %d or splits %d", max_m, splits);
   DK_REQUIRE(p.window >= 0 && p.chunk >= 0, "attention_rows_mma: bad window %d or chunk %d", p.window, p.chunk);
   DK_REQUIRE(p.gate == nullptr || p.gate_stride >= p.H, "attention_rows_mma: rows of %d gates do not hold %d heads", p.gate_stride, p.H);
   DK_REQUIRE(splits == 1 || part != nullptr, "attention_rows_mma: splits without scratch memory");
   DK_REQUIRE(p.row_q_start && p.row_q_len && p.row_pos_start && p.tok_row, "attention_rows_mma: the rows' arrays are missing");
   DK_REQUIRE((long long)p.rows * p.KV <= 65535, "attention_rows_mma: grid too large");
+  DK_REQUIRE((long long)p.num_pages * p.KV * p.ps < (1ll << 31), "attention_rows_mma: the cache of one layer has too many rows");
   int e;
   // a single token's heads: one warp; up to 64 query rows or a wide value: 16 rows a warp; else 32 rows a warp
   if (max_m <= 16) {

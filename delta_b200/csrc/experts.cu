@@ -242,6 +242,7 @@ router_kernel(const T* __restrict__ x, const T* __restrict__ w, float* __restric
     float acc[ROUTER_ROWS];
 #pragma unroll
     for (int q = 0; q < ROUTER_ROWS; ++q) acc[q] = 0.f;
+    // (rows behind the last one repeat it: no branch stands between the loads, so all of them are under way at once)
     if (VEC) {      // d is a multiple of 8 and the rows are 16-byte aligned: eight entries a load
 #pragma unroll 2
       for (int c = lane * 8; c < d; c += 256) {
@@ -249,20 +250,17 @@ router_kernel(const T* __restrict__ x, const T* __restrict__ w, float* __restric
         load8<T>(xr + c, xv);
 #pragma unroll
         for (int q = 0; q < ROUTER_ROWS; ++q) {
-          if (r0 + q < n_rows) {
-            float wv[8];
-            load8<T>(w + (size_t)(r0 + q) * d + c, wv);
+          float wv[8];
+          load8<T>(w + (size_t)min(r0 + q, n_rows - 1) * d + c, wv);
 #pragma unroll
-            for (int i = 0; i < 8; ++i) acc[q] = fmaf(xv[i], wv[i], acc[q]);
-          }
+          for (int i = 0; i < 8; ++i) acc[q] = fmaf(xv[i], wv[i], acc[q]);
         }
       }
     } else {
       for (int i = lane; i < d; i += 32) {
         const float xv = to_f32<T>(xr[i]);
 #pragma unroll
-        for (int q = 0; q < ROUTER_ROWS; ++q)
-          if (r0 + q < n_rows) acc[q] = fmaf(xv, to_f32<T>(w[(size_t)(r0 + q) * d + i]), acc[q]);
+        for (int q = 0; q < ROUTER_ROWS; ++q) acc[q] = fmaf(xv, to_f32<T>(w[(size_t)min(r0 + q, n_rows - 1) * d + i]), acc[q]);
       }
     }
 #pragma unroll
@@ -604,6 +602,51 @@ __global__ void experts_combine_kernel(const float* __restrict__ z, const float*
     out[(size_t)t * d + i] = from_f32<T>(a);
   }
 }
+
+// The same for a width that is a multiple of 8 with 16-byte aligned rows: eight columns a thread, several blocks a token.
+template <typename T, typename TX>
+__global__ void experts_combine_vec_kernel(const float* __restrict__ z, const float* __restrict__ weight, int top, const T* __restrict__ shared,
+                                           const float* __restrict__ gate_logit, int gate_stride, T* __restrict__ out, int d,
+                                           const TX* __restrict__ x, const int* __restrict__ choice, int identity_from) {
+  const int t = blockIdx.x, i = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
+  if (i >= d) return;
+  float a[8], s[8];
+#pragma unroll
+  for (int e = 0; e < 8; ++e) a[e] = s[e] = 0.f;
+  float gate = 0.f;
+  if (shared != nullptr) {
+    load8<T>(shared + (size_t)t * d + i, s);
+    gate = gate_logit != nullptr ? 1.f / (1.f + expf(-gate_logit[(size_t)t * gate_stride])) : 1.f;
+  }
+  const float* zt = z + (size_t)t * top * d + i;
+  if (x == nullptr) {
+#pragma unroll 4
+    for (int j = 0; j < top; ++j) {
+      float v[8];
+      load8<float>(zt + (size_t)j * d, v);
+      const float w = weight != nullptr ? weight[(size_t)t * top + j] : 1.f;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) a[e] = fmaf(w, v[e], a[e]);
+    }
+  } else {
+    float own[8];
+    load8<TX>(x + (size_t)t * d + i, own);
+#pragma unroll 4
+    for (int j = 0; j < top; ++j) {
+      const bool through = choice[(size_t)t * top + j] >= identity_from;
+      float v[8];
+      if (!through) load8<float>(zt + (size_t)j * d, v);      // (nothing was written at the place of such a choice)
+      const float w = weight != nullptr ? weight[(size_t)t * top + j] : 1.f;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) a[e] = fmaf(w, through ? own[e] : v[e], a[e]);
+    }
+  }
+  if (shared != nullptr) {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) a[e] = fmaf(gate, s[e], a[e]);
+  }
+  store8<T>(out + (size_t)t * d + i, a);
+}
 }  // namespace
 
 extern "C" int dk_experts_tile_rows() { return TILE_M; }
@@ -760,13 +803,22 @@ extern "C" int dk_experts_combine(const float* z, const float* weight, int top, 
   DK_REQUIRE(T_ > 0 && d > 0 && top > 0, "experts_combine: bad sizes T=%d d=%d top=%d", T_, d, top);
   DK_REQUIRE(x == nullptr || (choice != nullptr && identity_from >= 0), "experts_combine: an input is given without the choices");
   const int threads = d >= 1024 ? 256 : 128;
-#define LAUNCH(T, TX)                                                                                                             \
-  experts_combine_kernel<T, TX><<<T_, threads, 0, stream>>>(z, weight, top, (const T*)shared, gate_logit, gate_stride, (T*)out, d, \
-                                                            (const TX*)x, choice, identity_from)
+  auto aligned = [](const void* q) { return q == nullptr || ((uintptr_t)q % 16) == 0; };
+  const bool vec = d % 8 == 0 && d / 8 <= 65535 * 64 && aligned(z) && aligned(shared) && aligned(out) && aligned(x);
+  // few tokens: blocks of two warps, so that a token's columns are spread over several multiprocessors
+  const int vthreads = T_ <= 64 ? 64 : 128;
+  const dim3 vgrid(T_, (d / 8 + vthreads - 1) / vthreads);
+#define ARGS(T, TX) z, weight, top, (const T*)shared, gate_logit, gate_stride, (T*)out, d, (const TX*)x, choice, identity_from
+#define LAUNCH(T, TX)                                                                                 \
+  do {                                                                                                \
+    if (vec) experts_combine_vec_kernel<T, TX><<<vgrid, vthreads, 0, stream>>>(ARGS(T, TX));          \
+    else experts_combine_kernel<T, TX><<<T_, threads, 0, stream>>>(ARGS(T, TX));                      \
+  } while (0)
   if (dtype == DK_F32 && x_dtype == DK_F32) LAUNCH(float, float);
   else if (dtype == DK_F32 && x_dtype == DK_BF16) LAUNCH(float, __nv_bfloat16);
   else if (dtype == DK_BF16 && x_dtype == DK_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);
 #undef LAUNCH
+#undef ARGS
   else DK_REQUIRE(false, "experts_combine: unknown dtype %d", dtype);
   return dk_check_launch("experts_combine");
 }

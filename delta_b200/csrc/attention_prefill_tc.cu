@@ -32,8 +32,8 @@
 //   warp 11     issues P(j) V(j) when P(j) is written
 //
 // The queries' own keys were appended before this kernel runs, so a portion of a prompt
-// attends to the cache and to itself alike.  Pages past a row's last one are replaced by the
-// tile's first page: their scores are masked, and what is multiplied by the zeros is then
+// attends to the cache and to itself alike.  Pages past a row's last one, and pages before the first one that a
+// window still reaches (they were given back), are replaced by the tile's first page, or the pool's: their scores are masked, and what is multiplied by the zeros is then
 // finite.  Every wait is bounded; when one gives up the block records it, stores nothing,
 // frees its tensor memory and returns.
 #include "common.cuh"
@@ -81,7 +81,7 @@ __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
 // One piece of work: 128 queries of one head of one row.  Pieces are numbered with the head fastest, then the rows,
 // then the query tiles of each row from its latest (which has the most keys) to its first: from long to short.
 struct Piece {
-  int row, h, qt, nq, t0, pos0, last_pos, kt_first, n_tiles, last_page;
+  int row, h, qt, nq, t0, pos0, last_pos, kt_first, n_tiles, first_page, last_page;
   bool valid;
 };
 
@@ -100,6 +100,7 @@ __device__ __forceinline__ Piece piece_of(const DkAttnParams& p, int index, int 
   w.last_pos = w.pos0 + w.nq - 1;
   const int lo = (p.window > 0 && w.pos0 - p.window + 1 > 0) ? w.pos0 - p.window + 1 : 0;
   w.kt_first = lo / KT;
+  w.first_page = lo / p.ps;
   w.n_tiles = w.valid ? w.last_pos / KT - w.kt_first + 1 : 0;
   w.last_page = w.last_pos / p.ps;
   return w;
@@ -238,7 +239,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const 
         const int c = j & 1, ord = (c ? had1 : had0) + j / 2;     // the ord-th tile of its parity in this block
         const int lp = (w.kt_first + j) * ppt + lane;
         int page = -1;
-        if (lane < ppt && lp <= w.last_page && lp < p.max_pages) {
+        if (lane < ppt && lp >= w.first_page && lp <= w.last_page && lp < p.max_pages) {
           page = p.block_table[(size_t)w.row * p.max_pages + lp];
           if (page < 0 || page >= p.num_pages) {
             dk_report(p.err, DK_DEV_BAD_PAGE, w.row, lp, page);

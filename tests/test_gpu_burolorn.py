@@ -45,7 +45,8 @@ def make_runner(folder, which, dtype, num_pages=None, max_batch=4, max_seq_len=2
     return ModelRunner(folder, engine_config=cfg)
 
 
-CLOSE_CALL = 0.01      # a router's choice decided by less than this (in choice scores) may fall either way once the input is rounded to bfloat16
+CLOSE_CALL = 0.02      # a router's choice decided by less than this (in scores, or in a group's sum of two) may fall either way once the input is
+                       # rounded to bfloat16
 
 
 class Noise(list):

@@ -159,3 +159,25 @@ def test_scratch_addresses_stay_when_graphs_of_other_sizes_are_recorded(folders)
     want, _ = eager.step_and_sample([RowInput(s0, [5 + slots[0]], lens[0], [0], flags=1)])
     r.check_errors()
     assert (replayed[0] - want[0]).abs().max().item() <= bound_for(want[0], "bfloat16")
+
+
+def test_bfloat16_portions_behind_a_window(tmp_path):
+    """A layer with a window shorter than a key tile: later portions begin in tiles whose first pages were given back.  Long portions through
+    the tcgen05 kernel, against the whole prompt in one step."""
+    from delta_b200.config import EngineConfig
+    from delta_b200.engine.step import ModelRunner
+    from delta_b200.weights import write_random_model
+    import delta_b200.models  # noqa: F401
+    cfg = dict(helpers.tiny_config("D"), sliding_window=40, layer_types=["sliding_attention", "full_attention"])
+    folder = write_random_model(tmp_path / "windowed", cfg, 5, torch.bfloat16)
+    n = 460
+    toks = [helpers.random_tokens(n, cfg["vocab_size"], 3)]
+
+    def logits(steps):
+        r = ModelRunner(folder, engine_config=EngineConfig(max_batch=1, max_seq_len=512, page_size=16, num_pages=32, dtype="bfloat16"))
+        out = helpers.stack_positions(helpers.run_schedule(r, toks, steps), 0, n).double()
+        r.check_errors()
+        return out
+    a = logits([[(0, 0, n)]])
+    b = logits([[(0, p, min(76, n - p))] for p in range(0, n, 76)])
+    assert (a - b).pow(2).mean(dim=1).sqrt().max().item() <= 2e-2 * a.pow(2).mean().sqrt().item()

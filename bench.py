@@ -613,7 +613,8 @@ def design_workload(args, design: str) -> int:
             "latent_prepare": ((H * 192 + 320 + 320 + H * 64) * 2 * T * 4, 0),
             "rows_append": ((H + 2 * max(1, H // 4)) * 128 * 2 * T, 0),
             "gemm_nt_plain_batched": (0, 2 * T * H * (128 * 256 + 256 * 128) * 4),
-            "attention_rows_mma": (0, 4 * (2 * H * (320 + 256) * T * (T + 1) // 2) + 2 * H * 256 * (1024 * T - 1024 * 1023 // 2)),
+            "attention_rows_mma": (0, 4 * (2 * H * (320 + 256) * T * (T + 1) // 2)),      # the latent layers; the windowed one:
+            "attention_rows_tc": (0, 2 * H * 256 * (1024 * T - 1024 * 1023 // 2)),
         }
         def pibalorn_work():
             G, top, F = max(1, H // 4), 4, d // 2
@@ -627,7 +628,7 @@ def design_workload(args, design: str) -> int:
                 "experts_combine": ((top * d * 4 + 2 * d * 2) * T * n_moe, 0),
                 "decay_attention_chunked": (0, 2 * T * H * (2 * 128 * 128 + 16 * (128 + 128)) * n_lin),
                 "experts_gemm_tc": (0, 2 * T * top * 3 * d * F * n_moe),
-                "attention_rows_mma": (0, 4 * 128 * H * (T * (T + 1) // 2) * n_att),
+                "attention_rows_tc": (0, 4 * 128 * H * (T * (T + 1) // 2) * n_att),
             }
         if design == "pibalorn":
             work = pibalorn_work()
@@ -648,7 +649,7 @@ def design_workload(args, design: str) -> int:
                 "activation": (2 * top * F * 2 * T * n_moe, 0),
                 "experts_combine": ((top * d * 4 + d * 4) * T * n_moe, 0),
                 "experts_gemm_tc": (0, 2 * T * top * 2 * d * F * n_moe),
-                "attention_rows_mma": (0, 4 * 128 * H * seen * n_pair),
+                "attention_rows_tc": (0, 4 * 128 * H * seen * n_pair),
             }
         if design == "mufalix":
             work = mufalix_work()
@@ -714,7 +715,7 @@ def design_workload(args, design: str) -> int:
                 "experts_gather": (2 * top * d * 2 * T * n_moe, 0),
                 "experts_combine": ((top * d * 4 + 2 * d * 2) * T * n_moe, 0),
                 "experts_gemm_tc": (0, 2 * T * top * 3 * d * F * n_moe),
-                "attention_rows_mma": (0, 4 * 128 * H * (chunks * (n_att - n_full) + T * (T + 1) // 2 * n_full)),
+                "attention_rows_tc": (0, 4 * 128 * H * (chunks * (n_att - n_full) + T * (T + 1) // 2 * n_full)),
             }
         roletar_work = {
             "stream_norm": ((2 * S * d * 4 + 2 * d * 2) * T * (2 * runs), 0),
@@ -722,7 +723,8 @@ def design_workload(args, design: str) -> int:
             "rows_append": ((H + 2 * max(1, H // 4)) * 128 * 2 * T, 0),
             "gemm_nt_plain_batched": (0, 2 * T * H * (128 * 256 + 256 * 128) * 4),
             "library batched product": (0, 2 * T * H * (128 * 256 + 256 * 128) * 4),
-            "attention_rows_mma": (0, 4 * (2 * H * (320 + 256) * T * (T + 1) // 2) + 2 * H * 256 * (1024 * T - 1024 * 1023 // 2)),
+            "attention_rows_mma": (0, 4 * (2 * H * (320 + 256) * T * (T + 1) // 2)),      # the latent layers; the windowed one:
+            "attention_rows_tc": (0, 2 * H * 256 * (1024 * T - 1024 * 1023 // 2)),
             "selective_scan": ((4 * C + 2 * N) * 2 * T, 0),
             "conv_silu": (2 * C * 2 * T, 0),
         }

@@ -303,7 +303,7 @@ def test_convolution_norm_rotation_and_append(dtype, taps, H, KV, dk, dv, rot, i
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("taps,H,KV,dk,dv", [(4, 8, 2, 128, 64), (3, 8, 4, 64, 128), (2, 12, 2, 96, 32), (4, 8, 2, 64, 64), (4, 8, 2, 128, 128)])
+@pytest.mark.parametrize("taps,H,KV,dk,dv", [(4, 9, 3, 128, 64), (3, 8, 4, 64, 128), (2, 12, 2, 96, 32), (4, 8, 2, 64, 64), (4, 8, 2, 128, 128)])
 def test_convolution_over_long_portions(dtype, taps, H, KV, dk, dv):
     """Enough tokens for the tiles of several tokens a warp, whose edges fall inside rows, between them and on rows of one or two tokens."""
     check_conv_append(dtype, taps, H, KV, dk, dv, 32, False, [3, 1001, 1, 2, 1500], [0, 57, 9, 0, 700], ps=16)

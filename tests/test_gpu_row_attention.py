@@ -172,7 +172,7 @@ def test_one_key_that_matters(dtype, plain):
 
 
 @pytest.mark.parametrize("dtype,plain", KERNELS)
-@pytest.mark.parametrize("shape", [(6, 2, 64, 32), (8, 2, 128, 64), (4, 1, 48, 96), (2, 1, 96, 208), (32, 1, 64, 64)])
+@pytest.mark.parametrize("shape", [(6, 2, 64, 32), (12, 4, 128, 64), (4, 1, 48, 96), (2, 1, 96, 208), (32, 1, 64, 64)])
 def test_chunks_and_gates_of_heads(dtype, plain, shape):
     """Chunks that end inside tiles of queries and of keys, beside a gate per head: portions, single tokens (their keys split over several
     blocks), and both in one step."""
@@ -195,7 +195,7 @@ def test_the_chunks_first_key_and_the_one_before(dtype, plain):
 
 # ---- the tcgen05 kernel, also for portions shorter than those it is meant for ---------------------------------------------------
 
-TC_SHAPES = [(4, 2, 128, 128), (8, 2, 128, 64), (2, 1, 64, 128), (4, 4, 64, 64), (3, 1, 96, 80), (2, 1, 72, 104), (6, 3, 112, 64)]
+TC_SHAPES = [(4, 2, 128, 128), (12, 4, 128, 64), (2, 1, 64, 128), (4, 4, 64, 64), (3, 1, 96, 80), (2, 1, 72, 104), (6, 3, 112, 64)]
 
 
 @pytest.fixture
@@ -228,7 +228,7 @@ def test_tcgen05_portions(tc_everywhere, shape):
 
 
 def test_tcgen05_beside_single_tokens(tc_everywhere):
-    run_case("bfloat16", False, (8, 2, 128, 64), [(700, 1), (0, 150), (31, 1), (200, 90), (0, 1), (40, 2)], use_sink=True, gated=True, chunk=120, seed=6)
+    run_case("bfloat16", False, (12, 4, 128, 64), [(700, 1), (0, 150), (31, 1), (200, 90), (0, 1), (40, 2)], use_sink=True, gated=True, chunk=110, seed=6)
     run_case("bfloat16", False, (8, 2, 128, 128), [(0, 1), (700, 1), (600, 150)], seed=7)
 
 
